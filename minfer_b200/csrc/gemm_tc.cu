@@ -27,6 +27,11 @@
 // along K over a CLUSTER of CTAs, which add their partial tiles in rank order through
 // distributed shared memory (no atomics: reproducible), each finishing some of the tokens.
 //
+// Several products of one shape in one launch (mf_gemm_tc_grouped): the token rows lie packed group
+// after group, the weights are stacked, and a CTA finds its group and token tile from the groups'
+// first rows, which it reads on the device (rows routed to experts, for instance: nothing has to
+// come back to the host), or from a fixed number of rows a group.
+//
 // Every wait on an mbarrier is bounded: when it runs out the kernel sets
 // MF_STATUS_WAIT_TIMEOUT in the status word, stops issuing work, lets its copies land,
 // frees its tensor memory and returns.
@@ -79,6 +84,10 @@ struct GemmArgs {
     long long ldp;            // elements between consecutive tokens of prep_x
     float act_p, act_n;       // EPI_XIELU: the two coefficients of the activation
     int gate_act;             // EPI_SWIGLU: 0 silu, EPI_GATE_GELU_TANH
+    // grouped products: group g's token rows are group_first[g] .. group_first[g + 1] (device memory)
+    // or, with group_first null, g * group_rows .. (g + 1) * group_rows; its weight rows g * N ..
+    const int* group_first;
+    int n_groups, group_rows;
 };
 
 // an epilogue that is not linear in the accumulator cannot run on a K split's partial sums
@@ -305,10 +314,51 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& a, const uint32_t* r
 
 template <int NT> struct TmemCols { static constexpr int value = NT < 32 ? 32 : NT; };
 
-template <int NT, int STAGES>
+// The group and the first token of the `want`-th token tile (tiles numbered group after group), found
+// by one warp: 32 groups at a time, a prefix sum of their tiles.  `group` -1: there is no such tile.
+template <int NT>
+__device__ __forceinline__ void find_group_tile(const GemmArgs& a, int want, int lane, int& group, int& first,
+                                                int& end) {
+    group = -1; first = end = 0;
+    if (a.group_first == nullptr) {
+        const int per = (a.group_rows + NT - 1) / NT;
+        const int g = want / per;
+        if (g < a.n_groups) {
+            group = g;
+            first = g * a.group_rows + (want - g * per) * NT;
+            end = (g + 1) * a.group_rows;
+        }
+        return;
+    }
+    int before = 0;
+    for (int g0 = 0; g0 < a.n_groups; g0 += 32) {
+        const int g = g0 + lane;
+        const int lo = g < a.n_groups ? a.group_first[g] : 0, hi = g < a.n_groups ? a.group_first[g + 1] : 0;
+        int tiles = hi > lo ? (hi - lo + NT - 1) / NT : 0, sum = tiles;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int up = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += up;
+        }
+        const int start = before + sum - tiles;
+        const bool mine = want >= start && want < start + tiles;
+        const unsigned who = __ballot_sync(0xffffffffu, mine);
+        if (who != 0) {
+            const int src = __ffs(who) - 1;
+            group = g0 + src;
+            first = __shfl_sync(0xffffffffu, lo + (want - start) * NT, src);
+            end = __shfl_sync(0xffffffffu, hi, src);
+            return;
+        }
+        before += __shfl_sync(0xffffffffu, sum, 31);
+    }
+}
+
+template <int NT, int STAGES, bool GROUPED = false>
 __global__ void __launch_bounds__(128)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
-               const GemmArgs a) {
+               const GemmArgs args) {
+    GemmArgs a = args;
     constexpr int B_BYTES = NT * TILE_K * 2;
     constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
     constexpr int TMEM_COLS = TmemCols<NT>::value;
@@ -321,8 +371,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 
     pdl_launch_dependents();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int m0 = blockIdx.x * NT;                  // first token of this tile
+    int m0 = blockIdx.x * NT;                        // first token of this tile
     const int n0 = blockIdx.y * TILE_N;              // first row of W
+    int w0 = n0;                                     // ... in the stack of all groups' weights
+    if (GROUPED) {
+        pdl_wait();                                  // the groups' rows come from a kernel before
+        int group, end;
+        find_group_tile<NT>(a, blockIdx.x, lane, group, m0, end);
+        if (group < 0) return;                       // (every thread of the CTA finds the same)
+        a.M = end;
+        w0 = group * a.N + n0;
+    }
     const int split = blockIdx.z;
     const int kblocks = (a.K + TILE_K - 1) / TILE_K;
     const int kb0 = split * a.kblocks_per_split;
@@ -360,14 +419,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         for (int i = 0; i < pre; ++i) {
             const uint32_t full = smem_u32(&bars[i]);
             mbar_expect_tx(full, STAGE_BYTES);
-            tma_load_2d(smem_u32(smem + i * STAGE_BYTES), &map_w, (kb0 + i) * TILE_K, n0, full);
+            tma_load_2d(smem_u32(smem + i * STAGE_BYTES), &map_w, (kb0 + i) * TILE_K, w0, full);
         }
         // a CTA with only a few tiles beyond its ring asks for them in L2, so that the refill
         // after the first MMAs is not a trip to HBM on the step's critical path
         if (n_iter <= STAGES + 2)
             for (int i = pre; i < n_iter; ++i)
                 asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global.tile [%0, {%1, %2}];"
-                             ::"l"(&map_w), "r"((kb0 + i) * TILE_K), "r"(n0) : "memory");
+                             ::"l"(&map_w), "r"((kb0 + i) * TILE_K), "r"(w0) : "memory");
         pdl_wait();
         for (int i = 0; i < pre; ++i)
             tma_load_2d(smem_u32(smem + i * STAGE_BYTES) + A_BYTES, &map_x, (kb0 + i) * TILE_K, m0,
@@ -379,7 +438,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const uint32_t full = smem_u32(&bars[s]);
             mbar_expect_tx(full, STAGE_BYTES);
             const uint32_t dst = smem_u32(smem + s * STAGE_BYTES);
-            tma_load_2d(dst, &map_w, (kb0 + i) * TILE_K, n0, full);
+            tma_load_2d(dst, &map_w, (kb0 + i) * TILE_K, w0, full);
             tma_load_2d(dst + A_BYTES, &map_x, (kb0 + i) * TILE_K, m0, full);
         }
     } else {
@@ -782,6 +841,24 @@ static int weight_map(CUtensorMap* out, const void* ptr, int rows, int K, long l
     }
     *out = it->second;
     return 0;
+}
+
+template <int NT, int STAGES>
+static int launch_grouped(const CUtensorMap& mw, const CUtensorMap& mx, const GemmArgs& a, int tiles,
+                          cudaStream_t stream) {
+    constexpr int smem = STAGES * (A_BYTES + NT * TILE_K * 2) + 1024 + 256 + NT * 4;
+    static bool configured[64] = {false};
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return MF_ERR_UNSUPPORTED;
+    if (!configured[dev]) {
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<NT, STAGES, true>,
+                                             cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return (int)e;
+        configured[dev] = true;
+    }
+    mf_launch(gemm_tc_kernel<NT, STAGES, true>, dim3(tiles, (a.N + TILE_N - 1) / TILE_N, 1), dim3(128), smem,
+              stream, mw, mx, a);
+    return MF_LAUNCH_CHECK();
 }
 
 template <int NT, int STAGES>
@@ -1418,6 +1495,47 @@ extern "C" int mf_gemm_tc_gated(const void* x, long long ldx, const void* w, lon
     f.act_p = p0; f.act_n = p1;
     return gemm_tc_impl(x, ldx, w, ldw, nullptr, out, ldo, MF_DTYPE_BF16, M, N, K,
                         EPI_SWIGLU | ((gate_act & 0xff) << 8), nullptr, nullptr, status, &f, stream);
+}
+
+// Products of one shape over groups of token rows in one launch: rows of group g of x times the
+// transpose of w[g] (w: [groups][N][K], ldw elements between rows), into the same rows of `out`.
+// x holds `rows` rows in all.  The groups' rows: `group_first` [groups + 1] in device memory, or, null,
+// rows / groups each.  epi EPI_STORE, or EPI_SWIGLU with a gate's activation in its second byte and its
+// numbers p0, p1 (as mf_gemm_tc_gated).  Never split along K.
+extern "C" int mf_gemm_tc_grouped(const void* x, long long ldx, const void* w, long long ldw, void* out,
+                                  long long ldo, int out_dtype, int rows, int groups, const int* group_first,
+                                  int N, int K, int epi, float p0, float p1, unsigned* status,
+                                  cudaStream_t stream) {
+    const int gate_act = (epi >> 8) & 0xff;
+    epi &= 0xff;
+    if (rows <= 0 || groups <= 0 || N <= 0) return 0;
+    if (epi != EPI_STORE && epi != EPI_SWIGLU) return MF_ERR_ARGUMENT;
+    if (gate_act != 0 && (epi != EPI_SWIGLU || (gate_act != EPI_GATE_GELU_TANH && gate_act != EPI_GATE_CLAMPED_SWISH)))
+        return MF_ERR_ARGUMENT;
+    if (K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || (((uintptr_t)x | (uintptr_t)w) & 15)) return MF_ERR_UNSUPPORTED;
+    if (epi == EPI_SWIGLU && (out_dtype != MF_DTYPE_BF16 || N % 2 != 0)) return MF_ERR_UNSUPPORTED;
+    if (group_first == nullptr && rows % groups != 0) return MF_ERR_ARGUMENT;
+    if ((long long)groups * N > 0x7fffffffLL) return MF_ERR_UNSUPPORTED;
+    GemmArgs a = {};
+    a.out = out; a.status = status; a.ldo = ldo; a.M = rows; a.N = N; a.K = K; a.out_dtype = out_dtype;
+    a.kblocks_per_split = (K + TILE_K - 1) / TILE_K; a.epi = epi; a.gate_act = gate_act;
+    a.act_p = p0; a.act_n = p1;
+    a.group_first = group_first; a.n_groups = groups; a.group_rows = rows / groups;
+    const int mean = (rows + groups - 1) / groups;
+    const int nt = mean <= 16 ? 16 : mean <= 32 ? 32 : mean <= 64 ? 64 : 128;
+    // the most token tiles there can be: full ones, and a ragged one a group
+    const long long tiles = group_first ? (long long)rows / nt + (groups < rows ? groups : rows)
+                                        : (long long)groups * ((a.group_rows + nt - 1) / nt);
+    if (tiles > 0x7fffffffLL) return MF_ERR_UNSUPPORTED;
+    CUtensorMap mw, mx;
+    if (int e = weight_map(&mw, w, groups * N, K, ldw)) return e;
+    if (int e = make_map(&mx, x, rows, K, ldx, nt)) return e;
+    switch (nt) {
+        case 16: return launch_grouped<16, 6>(mw, mx, a, (int)tiles, stream);
+        case 32: return launch_grouped<32, 5>(mw, mx, a, (int)tiles, stream);
+        case 64: return launch_grouped<64, 4>(mw, mx, a, (int)tiles, stream);
+        default: return launch_grouped<128, 3>(mw, mx, a, (int)tiles, stream);
+    }
 }
 
 // out (+)= bias + sum over the K splits left in `partial` ([splits][M][N]) by a deferred

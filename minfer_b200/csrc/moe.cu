@@ -3,11 +3,12 @@
 //
 //   router_logits  the router's product in float32, a warp per (token, output)
 //   moe_route_scored   the router that scores with a softmax over all outputs (see there)
+//   moe_route_groups   the router that scores with a sigmoid and chooses within the best groups
 //   moe_route      per token: the `top` largest of its float32 router logits (ties: the lower
 //                  index), weights = softmax over the chosen logits only; a warp per token
 //   moe_up         hidden[t][k][f] = act(Wg_e x_t)[f] * (Wu_e x_t)[f] for token t's k-th expert e: a
 //                  block per (token, choice, tile of rows), a warp per row pair, x_t in shared memory
-//   moe_down       h[t][c] += sum_k w[t][k] (Wd_e hidden[t][k])[c], added into the float32 residual;
+//   moe_down       h[t][c] (+)= sum_k w[t][k] (Wd_e hidden[t][k])[c], added into the float32 residual;
 //                  one warp owns (t, c) and adds the choices in order, so the sum is reproducible
 //   moe_counts, moe_offsets, moe_place, moe_gather, moe_combine   for steps of many tokens the
 //                  (token, choice) pairs are grouped by expert and each expert runs as dense
@@ -180,6 +181,99 @@ extern "C" int mf_moe_route_scored(const float* logits, long long stride, const 
     return MF_LAUNCH_CHECK();
 }
 
+// Scores = sigmoid of each router output.  The experts form `groups` equal groups of neighbours; a
+// group's score is the sum of its two largest scores, and only experts of the `keep` best groups can
+// be chosen (groups 1: all).  The `top` largest scores among them are chosen (ties anywhere: the
+// lower index), with weights score / (sum of the chosen scores + 1e-20) * scale.  A warp per token.
+__global__ void __launch_bounds__(256)
+moe_route_groups_kernel(const float* __restrict__ logits, long long stride, int* __restrict__ idx,
+                        float* __restrict__ wts, int n_tokens, int experts, int top, int groups, int keep,
+                        float scale) {
+    pdl_prologue();
+    const int lane = threadIdx.x & 31;
+    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (t >= n_tokens) return;
+    const float* z = logits + (size_t)t * stride;
+    const int size = experts / groups;
+    unsigned long long allowed = ~0ull;                // bit g: group g may be chosen from
+    if (keep < groups) {
+        // lane g (and g + 32) holds the score of its group
+        float gs[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int g = lane + 32 * r;
+            if (g < groups) {
+                float a = -INFINITY, b = -INFINITY;
+                for (int i = 0; i < size; ++i) {
+                    const float s = 1.0f / (1.0f + expf(-z[g * size + i]));
+                    if (s > a) { b = a; a = s; } else if (s > b) b = s;
+                }
+                gs[r] = size > 1 ? a + b : a;
+            }
+        }
+        allowed = 0ull;
+        for (int k = 0; k < keep; ++k) {
+            float best = -INFINITY;
+            int best_g = 0x7fffffff;
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const int g = lane + 32 * r;
+                if (g < groups && !((allowed >> g) & 1ull) && gs[r] > best) { best = gs[r]; best_g = g; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+                const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+                if (ov > best || (ov == best && og < best_g)) { best = ov; best_g = og; }
+            }
+            if (best_g < groups) allowed |= 1ull << best_g;
+        }
+    }
+    int chosen_i[MOE_MAX_TOP];
+    float chosen_s[MOE_MAX_TOP];
+    float sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float best = -INFINITY;
+        int best_i = 0x7fffffff;
+        for (int e = lane; e < experts; e += 32) {
+            bool taken = keep < groups && !((allowed >> (e / size)) & 1ull);
+            for (int p = 0; p < k; ++p) taken |= chosen_i[p] == e;
+            const float s = 1.0f / (1.0f + expf(-z[e]));
+            if (!taken && (s > best || (s == best && e < best_i))) { best = s; best_i = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, best_i, o);
+            if (ov > best || (ov == best && oi < best_i)) { best = ov; best_i = oi; }
+        }
+        chosen_i[k] = best_i;
+        chosen_s[k] = best;
+        sum += best;
+    }
+    if (lane == 0) {
+        const float f = scale / (sum + 1e-20f);
+        for (int k = 0; k < top; ++k) {
+            // (logits that are not numbers compare with nothing: any expert in range, its weight is one too)
+            const bool found = chosen_i[k] < experts;
+            idx[(size_t)t * top + k] = found ? chosen_i[k] : k;
+            wts[(size_t)t * top + k] = found ? chosen_s[k] * f : z[k];
+        }
+    }
+}
+
+extern "C" int mf_moe_route_groups(const float* logits, long long stride, int* idx, float* wts,
+                                   int n_tokens, int experts, int top, int groups, int keep,
+                                   float scale, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (top < 1 || top > MOE_MAX_TOP || top > experts) return MF_ERR_UNSUPPORTED;
+    if (groups < 1 || groups > 64 || experts % groups != 0 || keep < 1 || keep > groups) return MF_ERR_UNSUPPORTED;
+    if (top > keep * (experts / groups)) return MF_ERR_ARGUMENT;
+    mf_launch(moe_route_groups_kernel, dim3((n_tokens + 7) / 8), dim3(256), 0, stream, logits, stride, idx,
+              wts, n_tokens, experts, top, groups, keep, scale);
+    return MF_LAUNCH_CHECK();
+}
+
 __device__ __forceinline__ float moe_dot(const float* w, const float* x, int n, int lane) {
     float s = 0.f;
     for (int i = lane; i < n; i += 32) s = fmaf(w[i], x[i], s);
@@ -246,7 +340,7 @@ template <typename TX, typename TW>
 __global__ void __launch_bounds__(256)
 moe_down_kernel(const TX* __restrict__ hidden, const TW* __restrict__ wd, const int* __restrict__ idx,
                 const float* __restrict__ wts, float* __restrict__ h, int width, int ff, int top,
-                int n_real, const TX* __restrict__ x) {
+                int n_real, const TX* __restrict__ x, int store) {
     pdl_launch_dependents();
     extern __shared__ float moe_hid[];             // [top][ff]
     const int t = blockIdx.x;                      // tokens along x, as the pairs above
@@ -264,7 +358,7 @@ moe_down_kernel(const TX* __restrict__ hidden, const TW* __restrict__ wd, const 
                 : warp_sum(moe_dot(wd + ((size_t)e * width + c) * ff, moe_hid + k * ff, ff, lane));
             sum = fmaf(wts[(size_t)t * top + k], d, sum);
         }
-        if (lane == 0) h[(size_t)t * width + c] += sum;
+        if (lane == 0) h[(size_t)t * width + c] = store ? sum : h[(size_t)t * width + c] + sum;
     }
 }
 
@@ -274,7 +368,8 @@ extern "C" int mf_moe_experts(const void* x, int x_dtype, const void* wg, const 
                               long long w_row, long long w_expert,
                               const void* wd, int w_dtype, const int* idx, const float* wts,
                               void* hidden, float* h, int n_tokens, int width, int ff, int top,
-                              int n_real, int act, float limit, float alpha, cudaStream_t stream) {
+                              int n_real, int act, float limit, float alpha, int store,
+                              cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top < 1 || top > MOE_MAX_TOP || (act != 0 && act != 2)) return MF_ERR_UNSUPPORTED;
     const size_t smem_up = (size_t)width * sizeof(float), smem_dn = (size_t)top * ff * sizeof(float);
@@ -289,7 +384,7 @@ extern "C" int mf_moe_experts(const void* x, int x_dtype, const void* wg, const 
                   (const TW*)wg, (const TW*)wu, w_row, w_expert, idx, (TX*)hidden, width, ff, top, n_real, \
                   act, limit, alpha); \
         mf_launch(moe_down_kernel<TX, TW>, grid_dn, dim3(256), smem_dn, stream, (const TX*)hidden, \
-                  (const TW*)wd, idx, wts, h, width, ff, top, n_real, (const TX*)x); \
+                  (const TW*)wd, idx, wts, h, width, ff, top, n_real, (const TX*)x, store); \
     } while (0)
     if (x_dtype == MF_DTYPE_F32 && w_dtype == MF_DTYPE_F32) MF_MOE(float, float);
     else if (x_dtype == MF_DTYPE_BF16 && w_dtype == MF_DTYPE_BF16) MF_MOE(__nv_bfloat16, __nv_bfloat16);
@@ -387,12 +482,12 @@ extern "C" int mf_moe_gather(const void* x, int dtype, const int* pairs, void* o
     return MF_LAUNCH_CHECK();
 }
 
-// h[t][:] += sum over the token's choices k, in order, of wts[t][k] * y[where[t * top + k]][:],
+// h[t][:] += (store: =) sum over the token's choices k, in order, of wts[t][k] * y[where[t * top + k]][:],
 // `where` the row of pair (t, k) in the experts' packed output; one thread owns an element
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ where,
                    const float* __restrict__ wts, float* __restrict__ h, int n_tokens, int width,
-                   int top) {
+                   int top, int store) {
     pdl_prologue();
     const long long total = (long long)n_tokens * width;
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total;
@@ -401,16 +496,16 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ where,
         float sum = 0.f;
         for (int k = 0; k < top; ++k)
             sum = fmaf(wts[(size_t)t * top + k], y[(size_t)where[(size_t)t * top + k] * width + c], sum);
-        h[i] += sum;
+        h[i] = store ? sum : h[i] + sum;
     }
 }
 
 extern "C" int mf_moe_combine(const float* y, const int* where, const float* wts, float* h,
-                              int n_tokens, int width, int top, cudaStream_t stream) {
+                              int n_tokens, int width, int top, int store, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     const long long total = (long long)n_tokens * width;
     const long long want = (total + 255) / 256, cap = (long long)mf_sm_count() * 16;
     mf_launch(moe_combine_kernel, dim3((unsigned)(want < cap ? want : cap)), dim3(256), 0, stream, y,
-              where, wts, h, n_tokens, width, top);
+              where, wts, h, n_tokens, width, top, store);
     return MF_LAUNCH_CHECK();
 }

@@ -1428,3 +1428,208 @@ extern "C" int mf_table_gate(const float* a, const void* table, int table_dtype,
 #undef MF_TG
     return MF_LAUNCH_CHECK();
 }
+
+// ------------------------------------------------------------------------------------
+// shift_mix: several mixes of a row with the row of the token before it,
+//     out[s][t][:] = x[t][:] + (x'[t][:] - x[t][:]) * mu[s][:],   s = 0 .. n_mix - 1,
+// x' the row of the sequence's previous token: in this step x[t - 1], for a row's first token
+// what `prev` [slots][width] (float32) holds for its slot.  `prev` takes the row's last x: by this
+// kernel where every row brings one token, by shift_keep afterwards otherwise (the block of a row's
+// first token may run after that of its last).
+// ------------------------------------------------------------------------------------
+template <typename T, int VEC> struct RowVec;
+template <> struct RowVec<float, 4> {
+    static __device__ __forceinline__ void load(const float* p, float* v) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+    }
+};
+template <> struct RowVec<__nv_bfloat16, 4> {
+    static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* v) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+        v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+    }
+};
+template <typename T> struct RowVec<T, 1> {
+    static __device__ __forceinline__ void load(const T* p, float* v) { v[0] = to_f32(*p); }
+};
+template <typename T, int VEC>
+__device__ __forceinline__ void row_store(T* p, const float* v) {
+    if (VEC == 4) Pack4<T>::store(p, v[0], v[1], v[2], v[3]);
+    else p[0] = from_f32<T>(v[0]);
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+shift_mix_kernel(const T* __restrict__ x, const float* __restrict__ mu, int n_mix, int n_tokens, int width,
+                 const int* __restrict__ token_row, const int* __restrict__ cu_seqlens,
+                 const int* __restrict__ slots, float* prev, T* __restrict__ out, int single) {
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int b = token_row[t];
+    const bool first = t == cu_seqlens[b];
+    float* kept = prev + (size_t)slots[b] * width;
+    pdl_wait();
+    const T* xr = x + (size_t)t * width;
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; i < width; i += gridDim.y * blockDim.x * VEC) {
+        float now[VEC], before[VEC];
+        RowVec<T, VEC>::load(xr + i, now);
+        if (first) RowVec<float, VEC>::load(kept + i, before);
+        else RowVec<T, VEC>::load(xr - width + i, before);
+        if (single) row_store<float, VEC>(kept + i, now);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) before[j] -= now[j];
+        for (int s = 0; s < n_mix; ++s) {
+            float m[VEC];
+            RowVec<float, VEC>::load(mu + (size_t)s * width + i, m);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) m[j] = fmaf(before[j], m[j], now[j]);
+            row_store<T, VEC>(out + ((size_t)s * n_tokens + t) * width + i, m);
+        }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+shift_keep_kernel(const T* __restrict__ x, int width, const int* __restrict__ cu_seqlens,
+                  const int* __restrict__ slots, float* __restrict__ prev) {
+    pdl_prologue();
+    const int b = blockIdx.x, last = cu_seqlens[b + 1] - 1;
+    if (last < cu_seqlens[b]) return;
+    for (int i = threadIdx.x; i < width; i += blockDim.x)
+        prev[(size_t)slots[b] * width + i] = to_f32(x[(size_t)last * width + i]);
+}
+
+extern "C" int mf_shift_mix(const void* x, int dtype, const float* mu, int n_mix, int n_tokens, int width,
+                            const int* token_row, const int* cu_seqlens, const int* slots, float* prev,
+                            void* out, int n_rows, int single, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_mix < 1 || width < 1 || n_rows < 1) return MF_ERR_ARGUMENT;
+    const bool vec = (width & 3) == 0 && (((uintptr_t)x | (uintptr_t)mu | (uintptr_t)prev | (uintptr_t)out) & 15) == 0;
+    const int per = vec ? 4 : 1;
+    int by = 1;
+    if (n_tokens < 2 * mf_sm_count()) by = (width + 256 * per - 1) / (256 * per);
+    dim3 grid(n_tokens, by), block(256);
+#define MF_SM(T, V) mf_launch(shift_mix_kernel<T, V>, grid, block, 0, stream, (const T*)x, mu, n_mix, n_tokens, \
+                              width, token_row, cu_seqlens, slots, prev, (T*)out, single)
+    if (dtype == MF_DTYPE_F32) { if (vec) MF_SM(float, 4); else MF_SM(float, 1); }
+    else if (dtype == MF_DTYPE_BF16) { if (vec) MF_SM(__nv_bfloat16, 4); else MF_SM(__nv_bfloat16, 1); }
+    else return MF_ERR_UNSUPPORTED;
+#undef MF_SM
+    if (!single) {
+        if (dtype == MF_DTYPE_F32)
+            mf_launch(shift_keep_kernel<float>, dim3(n_rows), block, 0, stream, (const float*)x, width, cu_seqlens, slots, prev);
+        else
+            mf_launch(shift_keep_kernel<__nv_bfloat16>, dim3(n_rows), block, 0, stream, (const __nv_bfloat16*)x, width,
+                      cu_seqlens, slots, prev);
+    }
+    return MF_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------
+// scaled_add: h[t][:] += a1[:] * y1[t][:] + a2[:] * y2[t][:], the end of a layer whose sublayers read
+// one norm and whose outputs each have a vector of factors.  A term is `y` [rows][width] (may be null)
+// plus the K splits of a product, `part` [n][rows][width] (may be null), added in split order; the
+// second term is left out when it has neither.  With `x_out` the norm that reads h next comes with
+// it: x_out[t][:] = h / sqrt(mean(h^2) + eps) * norm_w, in the type of the activations.
+// A block per row, the row in registers (width up to 4 * VEC * blockDim).
+// ------------------------------------------------------------------------------------
+struct ScaledTerm {
+    const float* y;
+    const float* part;
+    int n_part;
+    const float* scale;
+};
+
+template <int VEC>
+__device__ __forceinline__ void term_value(const ScaledTerm& s, size_t at, size_t split, float* v) {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = 0.0f;
+    if (s.y) RowVec<float, VEC>::load(s.y + at, v);
+#pragma unroll 4
+    for (int p = 0; p < s.n_part; ++p) {
+        float q[VEC];
+        RowVec<float, VEC>::load(s.part + (size_t)p * split + at, q);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v[j] += q[j];
+    }
+}
+
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(1024)
+scaled_add_kernel(float* __restrict__ h, ScaledTerm s1, ScaledTerm s2, int width, const float* __restrict__ norm_w,
+                  float eps, TO* __restrict__ x_out) {
+    pdl_prologue();
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * width, split = (size_t)gridDim.x * width;
+    const bool second = s2.y != nullptr || s2.n_part > 0;
+    float row[4][VEC];
+    float ss = 0.0f;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int i = (threadIdx.x + r * blockDim.x) * VEC;
+        if (i < width) {
+            float v[VEC], a[VEC];
+            RowVec<float, VEC>::load(h + base + i, row[r]);
+            term_value<VEC>(s1, base + i, split, v);
+            RowVec<float, VEC>::load(s1.scale + i, a);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[j] *= a[j];
+            if (second) {
+                float u[VEC];
+                term_value<VEC>(s2, base + i, split, u);
+                RowVec<float, VEC>::load(s2.scale + i, a);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) v[j] = fmaf(u[j], a[j], v[j]);
+            }
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                row[r][j] += v[j];
+                ss = fmaf(row[r][j], row[r][j], ss);
+            }
+            row_store<float, VEC>(h + base + i, row[r]);
+        }
+    }
+    if (x_out == nullptr) return;
+    ss = block_sum(ss, scratch);
+    const float f = 1.0f / sqrtf(ss / (float)width + eps);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int i = (threadIdx.x + r * blockDim.x) * VEC;
+        if (i < width) {
+            float w[VEC];
+            RowVec<float, VEC>::load(norm_w + i, w);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) w[j] = row[r][j] * f * w[j];
+            row_store<TO, VEC>(x_out + base + i, w);
+        }
+    }
+}
+
+extern "C" int mf_scaled_add(float* h, const float* y1, const float* part1, int n1, const float* scale1,
+                             const float* y2, const float* part2, int n2, const float* scale2, int n_rows,
+                             int width, const float* norm_w, float eps, void* x_out, int out_dtype,
+                             cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (width < 1 || scale1 == nullptr || (y1 == nullptr && n1 <= 0) || n1 < 0 || n2 < 0) return MF_ERR_ARGUMENT;
+    if ((n1 > 0 && part1 == nullptr) || (n2 > 0 && part2 == nullptr)) return MF_ERR_ARGUMENT;
+    if ((y2 != nullptr || n2 > 0) && scale2 == nullptr) return MF_ERR_ARGUMENT;
+    if (x_out != nullptr && norm_w == nullptr) return MF_ERR_ARGUMENT;
+    const ScaledTerm s1 = {y1, part1, n1, scale1}, s2 = {y2, part2, n2, scale2};
+    const uintptr_t ptrs = (uintptr_t)h | (uintptr_t)y1 | (uintptr_t)part1 | (uintptr_t)scale1 | (uintptr_t)y2 |
+                           (uintptr_t)part2 | (uintptr_t)scale2 | (uintptr_t)norm_w | (uintptr_t)x_out;
+    const bool vec = (width & 3) == 0 && (ptrs & 15) == 0;
+    const int per = vec ? 4 : 1;
+    if (width > 4 * 1024 * per) return MF_ERR_UNSUPPORTED;
+    // (a function of the width only: a row's sum never depends on the batch)
+    int threads = 32;
+    while (threads < 1024 && threads * 2 * per < width) threads <<= 1;
+#define MF_SA(T, V) mf_launch(scaled_add_kernel<T, V>, dim3(n_rows), dim3(threads), 0, stream, h, s1, s2, width, \
+                              norm_w, eps, (T*)x_out)
+    if (out_dtype == MF_DTYPE_F32) { if (vec) MF_SA(float, 4); else MF_SA(float, 1); }
+    else if (out_dtype == MF_DTYPE_BF16) { if (vec) MF_SA(__nv_bfloat16, 4); else MF_SA(__nv_bfloat16, 1); }
+    else return MF_ERR_UNSUPPORTED;
+#undef MF_SA
+    return MF_LAUNCH_CHECK();
+}

@@ -9,9 +9,10 @@
 //                     registers (d = lane + NS * i);
 //                     tokens are staged through shared memory RT_TC at a time by cp.async, the next
 //                     chunk travelling while this one is walked, four tokens' sums side by side.
-//   unit_norm_gate    each head's output divided by its root mean square (eps inside the root, no
-//                     weight), times silu or sigmoid of a gate read from the projection, times a
-//                     constant, written in the activation type.
+//   unit_norm_gate    each head's output, optionally divided by a number per (token, head) first,
+//                     divided by its root mean square (eps inside the root), times an optional
+//                     weight over all heads' values, times silu or sigmoid of a gate read from the
+//                     projection, times a constant, written in the activation type.
 // Tokens are packed row after row (row b: tokens cu_seqlens[b] .. cu_seqlens[b + 1]); a step may
 // bring any number of tokens per row.  All arithmetic is float32.
 #include "common.cuh"
@@ -212,7 +213,7 @@ template <typename TO>
 __global__ void __launch_bounds__(256)
 unit_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_width,
                       int gate_off, TO* __restrict__ out, long long items, int heads, int Dv, float eps,
-                      int act, float mul) {
+                      int act, float mul, const float* __restrict__ den, const float* __restrict__ weight) {
     pdl_prologue();
     const int lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -221,31 +222,37 @@ unit_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gat
     const int h = (int)(item - t * heads);
     const float* orow = o + (size_t)item * Dv;
     const float* grow = gate + (size_t)t * gate_width + gate_off + (size_t)h * Dv;
+    const float pre = den ? 1.0f / den[item] : 1.0f;
     float ss = 0.f;
-    for (int j = lane; j < Dv; j += 32) ss = fmaf(orow[j], orow[j], ss);
+    for (int j = lane; j < Dv; j += 32) {
+        const float x = orow[j] * pre;
+        ss = fmaf(x, x, ss);
+    }
     ss = warp_sum(ss);
-    const float inv = mul / sqrtf(ss / (float)Dv + eps);
+    const float inv = pre * (mul / sqrtf(ss / (float)Dv + eps));
     for (int j = lane; j < Dv; j += 32) {
         const float z = grow[j];
         const float sg = 1.0f / (1.0f + expf(-z));
-        out[(size_t)item * Dv + j] = from_f32<TO>(orow[j] * inv * (act == 0 ? z * sg : sg));
+        const float y = weight ? orow[j] * inv * weight[(size_t)h * Dv + j] : orow[j] * inv;
+        out[(size_t)item * Dv + j] = from_f32<TO>(y * (act == 0 ? z * sg : sg));
     }
 }
 
-// act 0: silu, 1: sigmoid
+// act 0: silu, 1: sigmoid; `den` [tokens][heads] and `weight` [heads * Dv] may be null
 extern "C" int mf_unit_norm_gate(const float* o, const float* gate, long long gate_width, int gate_off,
                                  void* out, int out_dtype, int n_tokens, int heads, int Dv, float eps,
-                                 int act, float mul, cudaStream_t stream) {
+                                 int act, float mul, const float* den, const float* weight,
+                                 cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (act != 0 && act != 1) return MF_ERR_ARGUMENT;
     const long long items = (long long)n_tokens * heads;
     dim3 grid((unsigned)((items + 7) / 8)), block(256);
     if (out_dtype == MF_DTYPE_F32)
         mf_launch(unit_norm_gate_kernel<float>, grid, block, 0, stream, o, gate, gate_width, gate_off,
-                  (float*)out, items, heads, Dv, eps, act, mul);
+                  (float*)out, items, heads, Dv, eps, act, mul, den, weight);
     else if (out_dtype == MF_DTYPE_BF16)
         mf_launch(unit_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, stream, o, gate, gate_width,
-                  gate_off, (__nv_bfloat16*)out, items, heads, Dv, eps, act, mul);
+                  gate_off, (__nv_bfloat16*)out, items, heads, Dv, eps, act, mul, den, weight);
     else return MF_ERR_UNSUPPORTED;
     return MF_LAUNCH_CHECK();
 }

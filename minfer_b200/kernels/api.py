@@ -127,6 +127,10 @@ def _sig_ops(lib: ctypes.CDLL) -> None:
                                 c_void_p]
     lib.mf_table_gate.argtypes = [c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
                                   c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+    lib.mf_shift_mix.argtypes = ([c_void_p, c_int, c_void_p] + [c_int] * 3 + [c_void_p] * 5 +
+                                 [c_int, c_int, c_void_p])
+    lib.mf_scaled_add.argtypes = ([c_void_p] + [c_void_p, c_void_p, c_int, c_void_p] * 2 +
+                                  [c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p])
 
 
 def _sig_gemm_simt(lib: ctypes.CDLL) -> None:
@@ -188,6 +192,9 @@ def _sig_gemm_tc(lib: ctypes.CDLL) -> None:
                                      c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                      c_void_p, c_int, c_int, c_float, c_void_p, c_longlong, c_void_p,
                                      c_void_p, c_void_p, c_void_p]
+    lib.mf_gemm_tc_grouped.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong,
+                                       c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float,
+                                       c_float, c_void_p, c_void_p]
     lib.mf_gemm_tc_xielu.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong,
                                      c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int,
                                      c_int, c_float, c_void_p, c_void_p]
@@ -224,7 +231,15 @@ def _sig_recurrent(lib: ctypes.CDLL) -> None:
 def _sig_retention(lib: ctypes.CDLL) -> None:
     lib.mf_retention_scan.argtypes = [c_void_p, c_void_p]
     lib.mf_unit_norm_gate.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int,
-                                      c_int, c_int, c_float, c_int, c_float, c_void_p]
+                                      c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p,
+                                      c_void_p]
+
+
+def _sig_outer_scan(lib: ctypes.CDLL) -> None:
+    lib.mf_wkv_scan.argtypes = [c_void_p, c_void_p]
+    lib.mf_mlstm_scan.argtypes = [c_void_p, c_void_p]
+    lib.mf_wkv_decay.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                 c_int, c_void_p]
 
 
 def _sig_mixer_prep(lib: ctypes.CDLL) -> None:
@@ -257,19 +272,21 @@ def _sig_moe(lib: ctypes.CDLL) -> None:
                                      c_void_p]
     lib.mf_moe_route_scored.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                                         c_int, c_int, c_void_p]
+    lib.mf_moe_route_groups.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int,
+                                        c_int, c_int, c_float, c_void_p]
     lib.mf_moe_experts.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_longlong,
                                    c_void_p, c_int, c_void_p,
                                    c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_float, c_float, c_void_p]
+                                   c_int, c_int, c_float, c_float, c_int, c_void_p]
     lib.mf_moe_counts.argtypes = [c_void_p, c_void_p, c_int, c_void_p]
     lib.mf_moe_place.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                  c_void_p]
     lib.mf_moe_gather.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
     lib.mf_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                   c_void_p]
+                                   c_int, c_void_p]
 
 
-_SIGNATURES = {"retention": _sig_retention, "delta_rule": _sig_delta_rule, "attention_talk": _sig_attention_talk, "moe": _sig_moe,
+_SIGNATURES = {"retention": _sig_retention, "outer_scan": _sig_outer_scan, "delta_rule": _sig_delta_rule, "attention_talk": _sig_attention_talk, "moe": _sig_moe,
                "attention_prefill_tc": _sig_attention_prefill_tc, "recurrent": _sig_recurrent,
                "mixer_prep": _sig_mixer_prep,
                "attention_sink": _sig_attention_sink,
@@ -625,6 +642,28 @@ def gemm_tc_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activatio
     _check(_lib("gemm_tc").mf_gemm_tc_gated(
         x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), m, n, k,
         GATE_CODES[activation], float(p0), float(p1), _i32(status, "status"), _stream()), "gemm_tc_gated")
+
+
+def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, first: Optional[torch.Tensor],
+                    status: torch.Tensor, activation: Optional[str] = None, p0: float = 0.0,
+                    p1: float = 0.0) -> None:
+    """Products of one shape over groups of rows, in one launch: the rows of group g of ``x`` [rows, K]
+    times w[g]^T (``w`` [groups, N, K]) into the same rows of ``out``.  ``first`` (int32 [groups + 1] on the
+    device): group g is rows first[g] .. first[g + 1]; None: rows / groups each.  ``activation``: the
+    weights' rows alternate gate, up and out is [rows, N / 2] bfloat16, as in ``gemm_tc_gated``."""
+    rows, k = x.shape
+    groups, n, kw = w.shape
+    cols = n if activation is None else n // 2
+    if (kw != k or out.shape != (rows, cols) or out.stride(1) != 1 or not w.is_contiguous()
+            or (first is not None and first.numel() != groups + 1) or (first is None and rows % groups != 0)):
+        raise KernelError("gemm_tc_grouped: shapes do not fit")
+    if not gemm_tc_supported(x, w[0]) or (activation is not None and out.dtype != torch.bfloat16):
+        raise KernelError("gemm_tc: operands must be bfloat16 with 16-byte aligned rows")
+    epi = EPI_STORE if activation is None else EPI_SWIGLU | (GATE_CODES[activation] << 8)
+    _check(_lib("gemm_tc").mf_gemm_tc_grouped(
+        x.data_ptr(), x.stride(0), w.data_ptr(), k, out.data_ptr(), out.stride(0), dtype_code(out.dtype), rows,
+        groups, _i32(first, "first"), n, k, epi, float(p0), float(p1), _i32(status, "status"), _stream()),
+        "gemm_tc_grouped")
 
 
 class RowScale:
@@ -983,6 +1022,10 @@ def qk_prepare(proj: torch.Tensor, positions: torch.Tensor, token_row: torch.Ten
            "qk_prepare")
 
 
+# ``q_rot_off`` of a ``qk_prepare`` whose query segment is not rotated (while its keys are)
+NO_ROTATION = -(1 << 20)
+
+
 class _HeadLinearArgs(ctypes.Structure):
     _fields_ = ([(n, c_void_p) for n in ("x", "w", "y", "gate")] +
                 [(n, c_longlong) for n in ("x_row", "y_row", "gate_row")] +
@@ -1265,10 +1308,29 @@ def moe_route_scored(logits: torch.Tensor, correction: Optional[torch.Tensor], i
         _f32(wts, "wts"), n, int(outputs), int(top), _stream()), "moe_route_scored")
 
 
+def moe_route_groups(logits: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, top: int, outputs: int,
+                     groups: int = 1, keep: int = 1, scale: float = 1.0) -> None:
+    """Per row of ``logits`` (float32 [tokens, >= outputs]; only the first ``outputs`` columns are the
+    router's): scores = sigmoid; the outputs form ``groups`` equal groups of neighbours, a group's
+    score is the sum of its two largest, and the ``top`` largest scores within the ``keep`` best
+    groups (ties: the lower index) go into ``idx``, score / (sum of the chosen + 1e-20) * ``scale``
+    into ``wts``."""
+    n = logits.shape[0]
+    if (idx.shape != (n, top) or wts.shape != (n, top) or logits.shape[1] < outputs
+            or logits.stride(1) != 1):
+        raise KernelError("moe_route_groups: shapes do not fit")
+    if not logits.is_cuda or logits.dtype != torch.float32:
+        raise KernelError("moe_route_groups: logits must be float32 on a CUDA device")
+    _check(_lib("moe").mf_moe_route_groups(
+        logits.data_ptr(), logits.stride(0), _i32(idx, "idx"), _f32(wts, "wts"), n, int(outputs),
+        int(top), int(groups), int(keep), float(scale), _stream()), "moe_route_groups")
+
+
 def moe_experts(x: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
                 idx: torch.Tensor, wts: torch.Tensor, hidden: torch.Tensor, h: torch.Tensor,
-                activation: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> None:
-    """h[t] += sum_k wts[t][k] Wd_e (silu(Wg_e x_t) * (Wu_e x_t)), e = idx[t][k]; with
+                activation: str = "silu", limit: float = 0.0, alpha: float = 1.0,
+                store: bool = False) -> None:
+    """h[t] += (``store``: =) sum_k wts[t][k] Wd_e (silu(Wg_e x_t) * (Wu_e x_t)), e = idx[t][k]; with
     ``activation`` "clamped_swish" an expert's hidden values are g' sigmoid(alpha g') (u' + 1),
     g' = min(g, limit), u' = clamp(u, -limit, limit).  A choice e >= the number of stacked experts
     names an expert without weights that returns the token's input: h[t] += wts[t][k] x_t.  ``w_gate`` and
@@ -1290,7 +1352,7 @@ def moe_experts(x: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor, w_dow
         _ptr(x, "x"), dtype_code(x.dtype), w_gate.data_ptr(), w_up.data_ptr(), w_gate.stride(1),
         w_gate.stride(0), _ptr(w_down, "w_down"), dtype_code(w_gate.dtype), _i32(idx, "idx"),
         _f32(wts, "wts"), _ptr(hidden, "hidden"), _f32(h, "h"), n, width, ff, top, int(experts),
-        EXPERT_ACTIVATIONS[activation], float(limit), float(alpha), _stream()),
+        EXPERT_ACTIVATIONS[activation], float(limit), float(alpha), 1 if store else 0, _stream()),
         "moe_experts", 2)
 
 
@@ -1322,13 +1384,15 @@ def moe_gather(x: torch.Tensor, pairs: torch.Tensor, out: torch.Tensor, top: int
                                      _stream()), "moe_gather")
 
 
-def moe_combine(y: torch.Tensor, where: torch.Tensor, wts: torch.Tensor, h: torch.Tensor) -> None:
-    """h[t] += sum_k wts[t][k] y[where[t][k]], the choices in order; y float32 rows."""
+def moe_combine(y: torch.Tensor, where: torch.Tensor, wts: torch.Tensor, h: torch.Tensor,
+                store: bool = False) -> None:
+    """h[t] += (``store``: =) sum_k wts[t][k] y[where[t][k]], the choices in order; y float32 rows."""
     n, top = where.shape
     if wts.shape != (n, top) or h.shape != (n, y.shape[1]):
         raise KernelError("moe_combine: shapes do not fit")
     _check(_lib("moe").mf_moe_combine(_f32(y, "y"), _i32(where, "where"), _f32(wts, "wts"),
-                                      _f32(h, "h"), n, y.shape[1], top, _stream()), "moe_combine")
+                                      _f32(h, "h"), n, y.shape[1], top, 1 if store else 0, _stream()),
+           "moe_combine")
 
 
 
@@ -1361,6 +1425,47 @@ def norm_add(h: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, e
     _check(_lib("ops").mf_norm_add(_f32(h, "h"), _f32(y, "y"), _f32(partial, "partial"), splits,
                                    _f32(bias, "bias"), _f32(weight, "weight"), n, width, float(eps),
                                    float(mult), _ptr(x_out, "x_out"), _stream()), "norm_add")
+
+
+def shift_mix(x: torch.Tensor, mu: torch.Tensor, token_row: torch.Tensor, cu_seqlens: torch.Tensor,
+              slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor, n_rows: int, single: bool) -> None:
+    """out[s][t] = x[t] + (x' - x[t]) * mu[s] for every mix s, x' the row of the sequence's token before
+    (``state`` [slots, width] float32 for a row's first token; it takes each row's last x).  ``mu``
+    float32 [mixes, width]; ``out`` [mixes, tokens, width] in the type of ``x``."""
+    n, width = x.shape
+    mixes = mu.shape[0]
+    if mu.shape != (mixes, width) or out.shape != (mixes, n, width) or out.dtype != x.dtype or state.shape[1] != width:
+        raise KernelError("shift_mix: shapes do not fit")
+    _check(_lib("ops").mf_shift_mix(
+        _ptr(x, "x"), dtype_code(x.dtype), _f32(mu, "mu"), mixes, n, width, _i32(token_row, "token_row"),
+        _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), _f32(state, "state"), _ptr(out, "out"),
+        int(n_rows), 1 if single else 0, _stream()), "shift_mix", 1 if single else 2)
+
+
+def scaled_add(h: torch.Tensor, first, second=None, norm_weight: Optional[torch.Tensor] = None,
+               eps: float = 0.0, x_out: Optional[torch.Tensor] = None) -> None:
+    """h[t] += scale1 * term1[t] + scale2 * term2[t].  ``first`` and ``second`` (None: left out) are
+    (y, partial, scale): ``y`` float32 [rows, width] or None, the K splits ``partial`` [splits, rows,
+    width] of a product or None, added in split order, ``scale`` float32 [width].  With ``x_out``
+    (the type of the activations): x_out = h / sqrt(mean(h^2) + eps) * norm_weight, the norm that reads
+    the new h next."""
+    n, width = h.shape
+    args = []
+    for term in (first, second):
+        if term is None:
+            args += [None, None, 0, None]
+            continue
+        y, partial, scale = term
+        if ((y is None and partial is None) or (y is not None and y.shape != h.shape) or scale.numel() != width
+                or (partial is not None and (partial.dim() != 3 or partial.shape[1:] != h.shape))):
+            raise KernelError("scaled_add: shapes do not fit")
+        args += [_f32(y, "y"), _f32(partial, "partial"), partial.shape[0] if partial is not None else 0,
+                 _f32(scale, "scale")]
+    if x_out is not None and (x_out.shape != h.shape or norm_weight is None or norm_weight.numel() != width):
+        raise KernelError("scaled_add: the norm does not fit the stream")
+    _check(_lib("ops").mf_scaled_add(_f32(h, "h"), *args, n, width, _f32(norm_weight, "norm_weight"), float(eps),
+                                     _ptr(x_out, "x_out"), dtype_code(x_out.dtype) if x_out is not None else F32,
+                                     _stream()), "scaled_add")
 
 
 UNARY_ACTIVATIONS = {"gelu": 0}
@@ -1521,18 +1626,96 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, proj: torch.Tensor, v_off: 
 
 
 def unit_norm_gate(o: torch.Tensor, gate: torch.Tensor, gate_off: int, out: torch.Tensor,
-                   heads: int, eps: float, activation: str = "silu", mul: float = 1.0) -> None:
-    """Each head of ``o`` (float32 [tokens, heads * Dv]) divided by its root mean square (eps inside
-    the root, no weight), times silu or sigmoid of the gate (columns gate_off .. of float32 rows),
-    times ``mul``."""
+                   heads: int, eps: float, activation: str = "silu", mul: float = 1.0,
+                   den: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None) -> None:
+    """Each head of ``o`` (float32 [tokens, heads * Dv]), divided by ``den`` (float32 [tokens, heads])
+    if that is given, divided by its root mean square (eps inside the root), times ``weight``
+    (float32 [heads * Dv]) if given, times silu or sigmoid of the gate (columns gate_off .. of
+    float32 rows), times ``mul``."""
     n = o.shape[0]
     dv = o.shape[1] // heads
+    if (den is not None and den.shape != (n, heads)) or (weight is not None and weight.numel() != heads * dv):
+        raise KernelError("unit_norm_gate: the divisors or the weight do not fit")
     if out.shape != o.shape or gate.shape[0] != n or gate_off + heads * dv > gate.shape[1]:
         raise KernelError("unit_norm_gate: shapes do not fit")
     _check(_lib("retention").mf_unit_norm_gate(
         _f32(o, "o"), _f32(gate, "gate"), gate.shape[1], int(gate_off), _ptr(out, "out"),
         dtype_code(out.dtype), n, heads, dv, float(eps), HEAD_GATES[activation], float(mul),
-        _stream()), "unit_norm_gate")
+        _f32(den, "den"), _f32(weight, "weight"), _stream()), "unit_norm_gate")
+
+
+class _OuterScanArgs(ctypes.Structure):
+    _fields_ = ([(n, c_void_p) for n in ("r", "k", "v", "w", "u", "gates", "i_bias", "f_bias", "state",
+                                         "maxima", "cu_seqlens", "slots", "out", "den")] +
+                [(n, c_longlong) for n in ("r_width", "k_width", "v_width", "w_width", "gate_width")] +
+                [(n, c_int) for n in ("r_off", "k_off", "v_off", "w_off", "i_off", "f_off", "n_rows",
+                                      "heads", "D", "Dv")] +
+                [("cap", c_float), ("r_scale", c_float)])
+
+
+def wkv_decay(t1: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t][c] = exp(-exp(w0[c] + sum_r w2t[r][c] tanh(t1[t][r]))), all float32: ``t1`` [tokens, rank]
+    (rows may be strided), ``w2t`` [rank, channels]."""
+    n, rank = t1.shape
+    channels = w0.numel()
+    if w2t.shape != (rank, channels) or out.shape != (n, channels) or t1.stride(1) != 1:
+        raise KernelError("wkv_decay: shapes do not fit")
+    if not t1.is_cuda or t1.dtype != torch.float32:
+        raise KernelError("wkv_decay: t1 must be float32 on a CUDA device")
+    _check(_lib("outer_scan").mf_wkv_decay(t1.data_ptr(), t1.stride(0), _f32(w2t, "w2t"), _f32(w0, "w0"),
+                                           _f32(out, "out"), n, rank, channels, _stream()), "wkv_decay")
+
+
+def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor,
+             state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
+             n_rows: int) -> None:
+    """Per (row, head), tokens one after another: out = S^T r + (r . (bonus k)) v, then
+    S <- diag(decay) S + k v^T.  ``r``, ``k``, ``decay`` float32 [tokens, heads * D], ``v`` and ``out``
+    [tokens, heads * Dv], ``bonus`` [heads, D]; S float32 in ``state`` [slots, heads, Dv, D]."""
+    n = r.shape[0]
+    _, heads, dv, d = state.shape
+    if (r.shape != (n, heads * d) or k.shape != r.shape or decay.shape != r.shape
+            or v.shape != (n, heads * dv) or out.shape != v.shape or bonus.numel() != heads * d):
+        raise KernelError("wkv_scan: shapes do not fit")
+    a = _OuterScanArgs()
+    a.r, a.k, a.v, a.w = _f32(r, "r"), _f32(k, "k"), _f32(v, "v"), _f32(decay, "decay")
+    a.u, a.state = _f32(bonus, "bonus"), _f32(state, "state")
+    a.cu_seqlens, a.slots, a.out = _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), _f32(out, "out")
+    a.r_width = a.k_width = a.w_width = heads * d
+    a.v_width = heads * dv
+    a.n_rows, a.heads, a.D, a.Dv = int(n_rows), heads, d, dv
+    a.r_scale = 1.0
+    _check(_lib("outer_scan").mf_wkv_scan(ctypes.addressof(a), _stream()), "wkv_scan")
+
+
+def mlstm_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off: int, f_off: int,
+               i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, q_scale: float,
+               state: torch.Tensor, maxima: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
+               out: torch.Tensor, den: torch.Tensor, n_rows: int) -> None:
+    """The matrix memory with exponential gates per (row, head), tokens one after another, from the
+    columns of the float32 rows ``proj``: q and k (heads of D), v (heads of Dv), the raw input and
+    forget gates (one per head).  ``out`` [tokens, heads * Dv] = S^T q (q times ``q_scale``) and
+    ``den`` [tokens, heads] = max(|n . q|, e^(-m)) + 1e-6, by which the output is still to be divided.
+    ``state`` float32 [slots, heads, Dv + 1, D]: S and, as the last column, n; ``maxima`` float32
+    [slots, heads, Dv + 1]: the running maximum, a copy per column."""
+    n = proj.shape[0]
+    _, heads, cols, d = state.shape
+    dv = cols - 1
+    if (out.shape != (n, heads * dv) or den.shape != (n, heads) or maxima.shape[1:] != (heads, cols)
+            or i_bias.numel() != heads or f_bias.numel() != heads
+            or max(max(q_off, k_off) + heads * d, v_off + heads * dv, max(i_off, f_off) + heads) > proj.shape[1]):
+        raise KernelError("mlstm_scan: shapes do not fit")
+    a = _OuterScanArgs()
+    a.r = a.k = a.v = a.gates = _f32(proj, "proj")
+    a.r_width = a.k_width = a.v_width = a.gate_width = proj.shape[1]
+    a.r_off, a.k_off, a.v_off, a.i_off, a.f_off = int(q_off), int(k_off), int(v_off), int(i_off), int(f_off)
+    a.i_bias, a.f_bias = _f32(i_bias, "i_bias"), _f32(f_bias, "f_bias")
+    a.state, a.maxima = _f32(state, "state"), _f32(maxima, "maxima")
+    a.cu_seqlens, a.slots = _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots")
+    a.out, a.den = _f32(out, "out"), _f32(den, "den")
+    a.n_rows, a.heads, a.D, a.Dv = int(n_rows), heads, d, dv
+    a.cap, a.r_scale = float(cap), float(q_scale)
+    _check(_lib("outer_scan").mf_mlstm_scan(ctypes.addressof(a), _stream()), "mlstm_scan")
 
 
 class _SelectiveArgs(ctypes.Structure):

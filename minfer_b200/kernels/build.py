@@ -43,6 +43,7 @@ LIBRARIES = {
     "attention_talk": ("attention_talk.cu", []),
     "moe": ("moe.cu", []),
     "retention": ("retention.cu", []),
+    "outer_scan": ("outer_scan.cu", []),
 }
 
 

@@ -3,12 +3,13 @@ from ..registry import register_part
 from .attention import Attention
 from .base import (Block, CacheRequest, CacheView, CallBinding, FeedForward, Mixer, Norm, Part,
                    PositionEncoding, StateRequest, StepContext)
-from .block import OutputNormBlock, PreNormBlock, TokenSide
+from .block import OutputNormBlock, ParallelBlock, PreNormBlock, TokenSide
 from .delta_rule import GatedDeltaRule
 from .latent_attention import LatentAttention
 from .linear import Linear
 from .mamba2 import Mamba2
 from .mlp import DenseMlp, GatedMlp
+from .mlstm import MLstm
 from .moe import RoutedExperts
 from .norm import RmsNorm
 from .parallel import ParallelMixer
@@ -20,6 +21,7 @@ from .selective_scan import SelectiveScan
 from .shift import TokenShift
 from .sink_attention import SinkAttention
 from .talking_attention import TalkingAttention
+from .wkv import Wkv
 from .stream import DepthAverage, EmbeddingNorm, LogitSoftcap, PassInjection
 
 register_part("norm", "rms_norm", RmsNorm, replace=True)
@@ -35,6 +37,8 @@ register_part("mixer", "talking_attention", TalkingAttention, replace=True)
 register_part("mixer", "retention", Retention, replace=True)
 register_part("mixer", "selective_scan", SelectiveScan, replace=True)
 register_part("mixer", "parallel", ParallelMixer, replace=True)
+register_part("mixer", "wkv", Wkv, replace=True)
+register_part("mixer", "mlstm", MLstm, replace=True)
 register_part("feed_forward", "gated_mlp", GatedMlp, replace=True)
 register_part("feed_forward", "dense_mlp", DenseMlp, replace=True)
 register_part("feed_forward", "routed_experts", RoutedExperts, replace=True)
@@ -46,4 +50,6 @@ register_part("model", "depth_average", DepthAverage, replace=True)
 register_part("block", "pre_norm", lambda layer, **options: PreNormBlock(layer, **options),
               replace=True)
 register_part("block", "output_norm", lambda layer, **options: OutputNormBlock(layer, **options),
+              replace=True)
+register_part("block", "parallel", lambda layer, **options: ParallelBlock(layer, **options),
               replace=True)

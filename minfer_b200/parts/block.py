@@ -12,7 +12,16 @@ from typing import Any, Dict, List, Mapping, Optional, Sequence
 import torch
 
 from ..config.base import LayerSpec
-from .base import Block, CallBinding, Part, StateRequest, StepContext, settle_pending
+from .base import Block, CallBinding, Part, Prepared, StateRequest, StepContext, settle_pending
+
+
+def sublayer_buffer(part, rows: int, width: int, device, ctx: StepContext) -> torch.Tensor:
+    """A float32 buffer of its own for a sublayer's output: zeros, or, for a part whose last product
+    can store (``stores_fresh_output``), memory that holds nothing yet."""
+    if getattr(part, "stores_fresh_output", False):
+        ctx.extras["fresh_output"] = True
+        return torch.empty((rows, width), dtype=torch.float32, device=device)
+    return torch.zeros((rows, width), dtype=torch.float32, device=device)
 
 
 class PreNormBlock(Block):
@@ -236,10 +245,7 @@ class OutputNormBlock(Block):
     def _output_buffer(part, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         """The buffer a sublayer adds its output into: zeros, or, for a part whose last product can
         store (``stores_fresh_output``), memory that holds nothing yet."""
-        if getattr(part, "stores_fresh_output", False):
-            ctx.extras["fresh_output"] = True
-            return torch.empty_like(h)
-        return torch.zeros_like(h)
+        return sublayer_buffer(part, h.shape[0], h.shape[1], h.device, ctx)
 
     def _add_normed(self, h: torch.Tensor, y: torch.Tensor, norm, ctx: StepContext) -> None:
         """h += mult * norm(y + whatever the sublayer's last product left pending)."""
@@ -272,3 +278,123 @@ class OutputNormBlock(Block):
             self._add_normed(h, y, self.feed_forward_norm, ctx)
         if self.side is not None:
             self.side.add(h, self._input(h, ctx), ctx)
+
+
+class ParallelBlock(Block):
+    """A block with one norm whose output both sublayers read, their outputs added together:
+
+        u = norm(h);   h += a1 * mixer(u) + a2 * ffn(u)                       (ffn optional)
+
+    ``layer_scale`` (names of two tensors [width], or None): the vectors a1 and a2; without it both
+    are 1.  Each sublayer writes a buffer of its own; one kernel then scales and adds both (with the K
+    splits their last products may have left) into the stream and, where the engine names the norm
+    that reads the stream next, norms it."""
+
+    capturable = True      # launches kernels only; safe inside a CUDA graph capture
+    accepts_pending = True     # a projection another block left pending is added by the norm
+
+    def __init__(self, layer: LayerSpec, layer_scale: Optional[Sequence[str]] = None, init_std: float = 0.1):
+        from ..registry import build_part
+        self.prefix = layer.prefix
+        self.norm = build_part("norm", layer.mixer_norm)
+        self.mixer = build_part("mixer", layer.mixer)
+        self.feed_forward = (build_part("feed_forward", layer.feed_forward)
+                             if layer.feed_forward is not None else None)
+        self.layer_scale = tuple(layer_scale) if layer_scale is not None else None
+        if self.layer_scale is not None and len(self.layer_scale) != 2:
+            raise ValueError("a layer scale names two tensors: the mixer's and the feed-forward's")
+        self.init_std = float(init_std)
+        self.width = int(layer.mixer_norm.params["size"])
+        self.scales: List[torch.Tensor] = []
+
+    def parts(self):
+        return tuple(p for p in (self.norm, self.mixer, self.feed_forward) if p is not None)
+
+    def libraries(self, dtype: torch.dtype) -> List[str]:
+        return ["ops", "moe"]
+
+    def _scale_names(self) -> List[str]:
+        if self.layer_scale is None:
+            return []
+        return [f"{self.prefix}{n}" for n in self.layer_scale[:2 if self.feed_forward is not None else 1]]
+
+    def tensor_specs(self, prefix: str = "") -> List:
+        from ..weights.spec import VECTOR, Init, TensorSpec
+        specs = PreNormBlock.tensor_specs(self, prefix)
+        return specs + [TensorSpec(n, (self.width,), VECTOR, Init(0.8, self.init_std)) for n in self._scale_names()]
+
+    def load(self, prefix: str, weights: Dict[str, torch.Tensor]) -> None:
+        PreNormBlock.load(self, prefix, weights)
+        names = self._scale_names()
+        if names:
+            self.scales = [weights[n] for n in names]
+        else:
+            like = next(iter(self.norm.export(self.prefix).values()))
+            one = torch.ones(self.width, dtype=torch.float32, device=like.device)
+            self.scales = [one, one]
+
+    def export(self, prefix: str = "") -> Dict[str, torch.Tensor]:
+        out = PreNormBlock.export(self, prefix)
+        out.update(zip(self._scale_names(), self.scales))
+        return out
+
+    def entry_norm(self):
+        return self.norm if self.norm.foldable() is not None else None
+
+    def _sublayer(self, part, x: torch.Tensor, ctx: StepContext, *args):
+        """Runs a sublayer on a buffer of its own: (the buffer or None, the K splits left pending or
+        None), whose sum is its output."""
+        ctx.extras.pop("prepare_for", None)
+        ctx.input_scale = None
+        n = x.shape[0]
+        y = sublayer_buffer(part, n, self.width, x.device, ctx)
+        part.forward_add(x, ctx, *args, y)
+        ctx.extras.pop("fresh_output", None)
+        pending = ctx.extras.pop("pending", None)
+        only = ctx.extras.pop("pending_only", False)
+        if pending is not None and pending.bias is not None:
+            from ..kernels import api as K
+            K.splitk_reduce(pending.partial, pending.bias, y, accumulate=not only)
+            return y, None
+        return (None if only else y), (pending.partial if pending is not None else None)
+
+    def mix(self, h: torch.Tensor, ctx: StepContext, binding: CallBinding) -> None:
+        prepared = ctx.extras.pop("prepared", None)
+        pending = ctx.extras.pop("pending", None)
+        if prepared is not None and prepared.norm is self.norm and prepared.scale is None:
+            x = prepared.x
+        elif pending is not None:
+            x = self.norm.forward_settling(h, pending, ctx.act_dtype)
+        else:
+            x = self.norm.forward(h, ctx.act_dtype)
+        ctx.extras["parallel"] = (x,) + self._sublayer(self.mixer, x, ctx, binding)
+
+    def feed(self, h: torch.Tensor, ctx: StepContext) -> None:
+        from ..kernels import api as K
+        x, y, partial = ctx.extras.pop("parallel")
+        rows = ctx.extras.get("kept_rows")
+        if rows is not None:               # the engine kept only these rows of h: the same of the rest
+            if partial is not None:
+                whole = torch.empty((x.shape[0], self.width), dtype=torch.float32, device=h.device) if y is None else y
+                K.splitk_reduce(partial, None, whole, accumulate=y is not None)
+                y, partial = whole, None
+            picked = torch.empty_like(h)
+            K.gather_rows(y, rows, picked)
+            y = picked
+            if self.feed_forward is not None:
+                kept = torch.empty((h.shape[0], x.shape[1]), dtype=x.dtype, device=h.device)
+                K.moe_gather(x, rows, kept, 1)
+                x = kept
+        second = None
+        if self.feed_forward is not None:
+            second = self._sublayer(self.feed_forward, x, ctx) + (self.scales[1],)
+        target = ctx.extras.get("next_norm")
+        fold = target.foldable() if target is not None else None
+        x_out = weight = None
+        eps = 0.0
+        if fold is not None and fold[2] == self.width:
+            weight, eps, _ = fold
+            x_out = torch.empty((h.shape[0], self.width), dtype=ctx.act_dtype, device=h.device)
+        K.scaled_add(h, (y, partial, self.scales[0]), second, weight, eps, x_out)
+        if x_out is not None:
+            ctx.extras["prepared"] = Prepared(x_out, None, target)

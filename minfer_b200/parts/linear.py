@@ -7,7 +7,7 @@ in the bfloat16 engine and is multiplied on the FP32 pipe.
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import Optional, Sequence
 
 import torch
 
@@ -104,3 +104,33 @@ class Linear:
         K.gemm_tc_fused(x, self.weight, self.bias, residual, K.EPI_ACCUM, gemm.status_word(x.device),
                         prep_x=xp, prep_weight=weight, prep_ssq=ssq)
         return Prepared(xp, K.RowScale(ssq, size, eps), norm)
+
+
+class GroupedLinear:
+    """Several projections of one shape, each on rows of its own: y[g] = x[g] W[g]^T, held stacked
+    [groups, out, in].  Few rows: one launch for all of them (a launch a projection is most of its
+    time there); many rows: a product each, on the kernel that is fastest for prompts."""
+
+    ONE_LAUNCH_MAX_ROWS = 255
+
+    def __init__(self, weights: Sequence[torch.Tensor]):
+        if len({t.dtype for t in weights}) != 1:
+            weights = [t.to(torch.float32) for t in weights]
+        self.weight = torch.stack(list(weights)).contiguous()
+        self.each = [Linear(w) for w in self.weight]
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        """``x`` [groups, rows, in] -> float32 [groups, rows, out]."""
+        from ..kernels import gemm
+        groups, n, width = x.shape
+        out = torch.empty((groups, n, self.weight.shape[1]), dtype=torch.float32, device=x.device)
+        if n == 0:
+            return out
+        flat = x.view(groups * n, width)
+        if (n <= self.ONE_LAUNCH_MAX_ROWS and x.dtype == torch.bfloat16 and gemm.use_tensor_cores()
+                and K.gemm_tc_supported(flat, self.weight[0])):
+            K.gemm_tc_grouped(flat, self.weight, out.view(groups * n, -1), None, gemm.status_word(x.device))
+        else:
+            for g, linear in enumerate(self.each):
+                linear.forward(x[g], torch.float32, out=out[g])
+        return out

@@ -12,6 +12,10 @@ Options for designs that route otherwise (each a parameter):
                             largest s + correction are chosen (``correction_name``: a tensor of one
                             number per output; None: none); the weights are the chosen s themselves,
                             not renormalized
+    scoring "sigmoid_groups" scores s = sigmoid(z); the experts form ``groups`` equal groups of neighbours,
+                            a group's score is the sum of its two largest s, and the ``top`` largest s
+                            within the ``keep_groups`` best groups are chosen; their weights are
+                            s / (sum of the chosen s + 1e-20) * ``weight_scale``
     identity                the last ``identity`` router outputs (beyond the ``n_experts`` experts with
                             weights) stand for experts that return the token's input: weight * u
     activation "clamped_swish"   y = g' sigmoid(1.702 g') (u' + 1), g' = min(Wg u, limit),
@@ -26,10 +30,12 @@ load ([experts, ff, width] and [experts, width, ff]).
 
 Two ways through a step.  Few tokens (decoding; always inside a CUDA graph capture): one kernel
 per half, a block per (token, choice), the expert's rows read by index; nothing is read back.  Many
-tokens: the (token, choice) pairs are grouped by expert on the device, the offsets come back to the
-host (one small read), and each expert runs as two dense products over its rows, the gate's
-activation in the first one's epilogue; the weighted rows are then added into the residual token by
-token, the choices in order, so the sum does not depend on the batch.
+tokens: the (token, choice) pairs are grouped by expert on the device, and every expert runs as two
+dense products over its rows, the gate's activation in the first one's epilogue; the weighted rows are
+then added into the residual token by token, the choices in order, so the sum does not depend on the
+batch.  On the tensor cores the two products of all experts are two launches, whose blocks read the
+experts' offsets themselves; otherwise the offsets come back to the host (one small read) for a
+product per expert.
 """
 from __future__ import annotations
 
@@ -42,6 +48,7 @@ from ..kernels import api as K
 from ..weights.spec import MATRIX, VECTOR, Init, TensorSpec
 from .base import FeedForward, StepContext, settle_pending
 from .linear import Linear
+from .sink_attention import project_out
 
 # steps of up to this many tokens run the per-token kernels
 PER_TOKEN_MAX = int(os.environ.get("MINFER_B200_MOE_PER_TOKEN_MAX", "48"))
@@ -49,6 +56,7 @@ PER_TOKEN_MAX = int(os.environ.get("MINFER_B200_MOE_PER_TOKEN_MAX", "48"))
 
 class RoutedExperts(FeedForward):
     capturable = True      # the per-token path launches kernels only; captures always take it
+    stores_fresh_output = True     # answers ``ctx.extras["fresh_output"]`` (see ``project_out``)
 
     def libraries(self, dtype: torch.dtype) -> List[str]:
         return ["ops", "moe", "gemm_simt"] + (["gemm_tc"] if dtype == torch.bfloat16 else [])
@@ -58,16 +66,25 @@ class RoutedExperts(FeedForward):
                  router_bias_name: Optional[str] = "mlp.router.b",
                  expert_name: str = "mlp.e{e}", init_std: float = 0.02, router_std: float = 0.5,
                  scoring: str = "softmax_top", correction_name: Optional[str] = None,
-                 identity: int = 0, limit: float = 0.0, shared: Optional[dict] = None):
+                 identity: int = 0, limit: float = 0.0, shared: Optional[dict] = None,
+                 groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0):
         if activation not in K.EXPERT_ACTIVATIONS:
             raise ValueError(f"the experts' activation is one of {sorted(K.EXPERT_ACTIVATIONS)}, got "
                              f"{activation!r}")
-        if scoring not in ("softmax_top", "softmax_all"):
-            raise ValueError(f"scoring is softmax_top or softmax_all, got {scoring!r}")
+        if scoring not in ("softmax_top", "softmax_all", "sigmoid_groups"):
+            raise ValueError(f"scoring is softmax_top, softmax_all or sigmoid_groups, got {scoring!r}")
+        if scoring == "sigmoid_groups":
+            if not 1 <= groups <= 64 or n_experts % groups != 0 or not 1 <= keep_groups <= groups:
+                raise ValueError(f"{n_experts} experts do not form {groups} groups (up to 64) of which "
+                                 f"{keep_groups} are kept")
+            if top > keep_groups * (n_experts // groups):
+                raise ValueError(f"{keep_groups} groups of {n_experts // groups} experts do not hold {top} to choose")
+            if correction_name is not None:
+                raise ValueError("the scoring sigmoid_groups takes no correction")
         if identity < 0 or (identity > 0 and scoring != "softmax_all"):
             raise ValueError("experts without weights need the scoring softmax_all")
-        if shared is not None and scoring != "softmax_all":
-            raise ValueError("a shared expert needs the scoring softmax_all")
+        if shared is not None and scoring == "softmax_top":
+            raise ValueError("a shared expert needs the scoring softmax_all or sigmoid_groups")
         if activation == "clamped_swish" and not limit > 0.0:
             raise ValueError("the clamped activation needs a positive limit")
         if not 1 <= top <= n_experts + identity:
@@ -80,6 +97,7 @@ class RoutedExperts(FeedForward):
         self.top = int(top)
         self.activation = activation
         self.scoring, self.correction_name = scoring, correction_name
+        self.groups, self.keep_groups, self.weight_scale = int(groups), int(keep_groups), float(weight_scale)
         self.identity = int(identity)
         self.n_outputs = self.n_experts + self.identity          # what the router chooses among
         self.limit = float(limit)
@@ -203,7 +221,9 @@ class RoutedExperts(FeedForward):
     # ---- the step -----------------------------------------------------------------------
     def forward_add(self, x: torch.Tensor, ctx: StepContext, residual: torch.Tensor) -> None:
         ctx.extras.pop("prepare_for", None)
-        settle_pending(ctx, residual)              # the experts add into the complete stream
+        fresh = ctx.extras.pop("fresh_output", False)
+        if not fresh:
+            settle_pending(ctx, residual)          # the experts add into the complete stream
         n, dev = x.shape[0], x.device
         if n == 0:
             return
@@ -217,14 +237,17 @@ class RoutedExperts(FeedForward):
         wts = torch.empty((n, self.top), dtype=torch.float32, device=dev)
         if self.scoring == "softmax_all":
             K.moe_route_scored(logits, self.correction, idx, wts, self.top, self.n_outputs)
+        elif self.scoring == "sigmoid_groups":
+            K.moe_route_groups(logits, idx, wts, self.top, self.n_outputs, self.groups, self.keep_groups,
+                               self.weight_scale)
         else:
             K.moe_route(logits, idx, wts, self.top)
         if self.per_token_fits and (n <= PER_TOKEN_MAX or torch.cuda.is_current_stream_capturing()):
             hidden = torch.empty((n, self.top, self.intermediate_size), dtype=x.dtype, device=dev)
             K.moe_experts(x, self.w_gate, self.w_up, self.w_down, idx, wts, hidden, residual,
-                          self.activation, self.limit, self.alpha)
+                          self.activation, self.limit, self.alpha, store=fresh)
         else:
-            self._grouped(x, idx, wts, residual)
+            self._grouped(x, idx, wts, residual, fresh)
         if self.shared is not None:
             # act(gate, up) * sigmoid(the router product's extra column), then down into the stream
             from ..kernels import gemm
@@ -241,10 +264,14 @@ class RoutedExperts(FeedForward):
                 gu = self.shared_gate_up.forward(x, torch.float32)
                 K.gated_act(gu, act, self.activation, float(self.shared["limit"]), self.alpha,
                             row_gate=row_gate, interleaved=self.shared_interleaved)
-            self.shared_down.forward(act, torch.float32, out=residual, accumulate=True)
+            if fresh:
+                # (the block that owns the buffer adds the K splits of a small product itself)
+                project_out(self.shared_down, act, ctx, residual)
+            else:
+                self.shared_down.forward(act, torch.float32, out=residual, accumulate=True)
 
     def _grouped(self, x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor,
-                 residual: torch.Tensor) -> None:
+                 residual: torch.Tensor, store: bool) -> None:
         from ..kernels import gemm
         n, dev = x.shape[0], x.device
         ff, width, top = self.intermediate_size, self.hidden_size, self.top
@@ -255,7 +282,6 @@ class RoutedExperts(FeedForward):
         where = torch.empty((n, top), dtype=torch.int32, device=dev)
         K.moe_counts(idx, counts)
         K.moe_place(idx, counts, offsets, order, where)
-        first = offsets.tolist()                   # the one read of the step: rows per expert
         xg = torch.empty((n_pairs, width), dtype=x.dtype, device=dev)
         K.moe_gather(x, order, xg, top)
         act = torch.empty((n_pairs, ff), dtype=x.dtype, device=dev)
@@ -263,6 +289,14 @@ class RoutedExperts(FeedForward):
         fused = (self.w_gate_up.dtype == torch.bfloat16 and x.dtype == torch.bfloat16
                  and gemm.use_tensor_cores()
                  and K.gemm_tc_supported(xg, self.w_gate_up[0]))
+        if (fused and self.identity == 0 and self.w_down.dtype == torch.bfloat16
+                and K.gemm_tc_supported(act, self.w_down[0])):
+            status = gemm.status_word(dev)
+            K.gemm_tc_grouped(xg, self.w_gate_up, act, offsets, status, self.activation, self.limit, self.alpha)
+            K.gemm_tc_grouped(act, self.w_down, y, offsets, status)
+            K.moe_combine(y, where, wts, residual, store=store)
+            return
+        first = offsets.tolist()                   # the one read of the step: rows per expert
         for e in range(self.n_outputs):
             lo, hi = first[e], first[e + 1]
             if hi <= lo:
@@ -289,4 +323,4 @@ class RoutedExperts(FeedForward):
                     Linear(self.w_up[e]).forward(xe, torch.float32, out=gu[:, ff:])
                     K.gated_act(gu, ae, self.activation, self.limit, self.alpha)
             Linear(self.w_down[e]).forward(ae, torch.float32, out=y[lo:hi])
-        K.moe_combine(y, where, wts, residual)
+        K.moe_combine(y, where, wts, residual, store=store)
