@@ -1303,6 +1303,297 @@ def workload_zanelorn(args) -> int:
     return 0
 
 
+# ------------------------------------------------------------------------------------------
+# --workload pikavik: the Pikavik design beside the Qwen2 decoder at equal width and layers
+# ------------------------------------------------------------------------------------------
+# (name, width, latent attention heads, feed-forward width of Qwen2, mLSTM heads): six layers, WKV,
+# mLSTM and latent attention in turn, a routed feed-forward in each: 32 experts of a quarter of the
+# dense feed-forward in 8 groups of which 5 are kept, 4 experts a token and a shared one.  WKV heads of
+# 64 over the whole width; mLSTM keys of 128 with values of 256; attention keys of 64 + 64 rotated and
+# values of 128 from a latent of 512, queries through a latent of 3/8 of the width
+PIKAVIK_SIZES = [("w2048", 2048, 16, 5632, 8), ("w4096", 4096, 32, 11264, 16)]
+PIKAVIK_LAYERS = 6
+PIKAVIK_RANK = 512
+
+
+def pikavik_config(width, heads, ff, lstm_heads, vocab):
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0},
+           "router": {"experts": 32, "top": 4, "scale": 2.5, "groups": {"count": 8, "keep": 5}},
+           "shared": {"ff": ff // 4, "limit": 7.0}}
+    mixers = [{"type": "wkv", "mixer": {"heads": width // 64, "dim": 64, "decay_rank": 64}},
+              {"type": "mlstm", "mixer": {"heads": lstm_heads, "dim": 128, "vdim": 256, "gate_cap": 15.0}},
+              {"type": "latent_attention",
+               "mixer": {"heads": heads, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": PIKAVIK_RANK,
+                         "q_rank": 3 * width // 8, "scale": 128 ** -0.5, "rot": {"base": 100000.0, "dims": 64}}}]
+    return {"architecture": "Pikavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [dict(mixers[i % 3], mlp=moe) for i in range(PIKAVIK_LAYERS)]}
+
+
+def pikavik_prefill_flops(cfg, tokens):
+    """Matrix-product flops of one whole prompt (head on the last row only; the experts a token uses,
+    not all), the attention of the visible keys, and the recurrences (per token and state element:
+    decay, update and read-out)."""
+    w, n = cfg["width"], tokens
+    flops = 0.0
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer["mlp"]
+        pairs = 0.0
+        if layer["type"] == "wkv":
+            h, d = m["heads"], m["dim"]
+            per_token = 2 * w * 5 * h * d + 2 * m["decay_rank"] * (w + h * d) + 6 * h * d * d
+        elif layer["type"] == "mlstm":
+            h, d, dv = m["heads"], m["dim"], m["vdim"]
+            per_token = 2 * w * (2 * h * d + 3 * h * dv + 2 * h) + 6 * h * d * dv
+        else:
+            h, d, r, dv, rank, qr = (m[x] for x in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+            per_token = (2 * w * (qr + rank + r) + 2 * qr * h * (d + r) + 2 * rank * h * (d + dv)
+                         + 2 * w * h * dv)
+            pairs = h * 2 * (d + r + dv) * n * (n + 1) / 2
+        per_token += mlp["router"]["top"] * 6 * w * mlp["expert"]["ff"] + 2 * w * (mlp["router"]["experts"] + 1)
+        per_token += 6 * w * mlp["shared"]["ff"]
+        flops += per_token * n + pairs
+    return flops + 2 * w * cfg["vocab"]
+
+
+def pikavik_decode_bytes(model, cfg, batch, context_tokens):
+    """Bytes a decode step must read: the weights it touches (of each layer's experts as many as
+    ``batch`` tokens choose on average if every expert is as likely), one row of the embedding per
+    sequence, the latent vectors of the context and the recurrent states (read and written)."""
+    total = model.parameter_bytes()
+    w = cfg["width"]
+    total -= cfg["vocab"] * w * 2
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer["mlp"]
+        experts, top = mlp["router"]["experts"], mlp["router"]["top"]
+        total -= experts * (1.0 - top / experts) ** batch * 3 * w * mlp["expert"]["ff"] * 2
+        if layer["type"] == "wkv":
+            total += batch * 2 * m["heads"] * m["dim"] ** 2 * 4
+        elif layer["type"] == "mlstm":
+            total += batch * 2 * m["heads"] * m["dim"] * (m["vdim"] + 1) * 4
+        else:
+            total += batch * context_tokens * (m["kv_rank"] + m["rot_dim"]) * 2
+    return total
+
+
+def pikavik_kernels(torch, K, pk, width, heads, ff, lstm_heads, tokens=2048, batch=8):
+    """The design's own kernels alone (median of 20, L2 flushed before each): device time and the
+    fraction of the copy bandwidth (or of the product peak) their algorithmic bytes (flops) reach,
+    each beside the like kernel of another design at equal sizes."""
+    from minfer_b200.parts.base import CacheView, StepContext
+    from minfer_b200.parts.sink_attention import ScoreSpec, scored_attention
+    dev = "cuda:0"
+    bw = pk["hbm_gbs"] * 1e9
+    peak = pk["bf16_tflops"] * 1e12
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bf = torch.bfloat16
+    out = {}
+
+    def timed(name, fn, nbytes=None, flops=None):
+        ms = _median_ms(torch, fn, 20, flush)
+        out[name] = {"us": round(ms * 1e3, 1)}
+        if nbytes is not None:
+            out[name]["frac_of_copy"] = round(nbytes / (ms * 1e-3) / bw, 4)
+        if flops is not None:
+            out[name]["frac_of_product_peak"] = round(flops / (ms * 1e-3) / peak, 4)
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    def rnd(*shape):
+        return torch.randn(*shape, device=dev)
+
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    vec = torch.ones(width, device=dev)
+    for label, n, rows in (("prompt", tokens, 1), ("decode", batch, batch)):
+        per = n // rows
+        cu, slots = i32([per * b for b in range(rows + 1)]), i32(list(range(rows)))
+        positions = i32([tokens + (t % per) if label == "decode" else t for t in range(n)])
+        token_row = i32([t // per for t in range(n)])
+        single = label == "decode"
+        # ---- WKV: mixes, decays, scan, beside the state-space and retention scans ------------------------
+        H, D = width // 64, 64
+        x = rnd(n, width).to(bf)
+        mixes = torch.empty(5, n, width, dtype=bf, device=dev)
+        mu, prev = torch.rand(5, width, device=dev), torch.zeros(rows, width, device=dev)
+        timed(f"shift_mix_{label}", lambda: K.shift_mix(x, mu, token_row, cu, slots, prev, mixes, rows, single),
+              nbytes=n * width * 12)
+        t1, w2t, w0 = rnd(n, 64), rnd(64, H * D) * 0.1, rnd(H * D) - 2
+        decay = torch.empty(n, H * D, device=dev)
+        timed(f"wkv_decay_{label}", lambda: K.wkv_decay(t1, w2t, w0, decay), nbytes=n * (64 + H * D) * 4 + 64 * H * D * 4)
+        r, k, v, u = rnd(n, H * D), rnd(n, H * D) * 0.1, rnd(n, H * D), rnd(H, D)
+        state, o = torch.zeros(rows, H, D, D, device=dev), torch.empty(n, H * D, device=dev)
+        timed(f"wkv_scan_{label}", lambda: K.wkv_scan(r, k, v, decay, u, state, cu, slots, o, rows),
+              nbytes=n * 5 * H * D * 4 + rows * 2 * H * D * D * 4)
+        # ---- mLSTM beside retention of the same keys and values ---------------------------------------------
+        H, D, Dv = lstm_heads, 128, 256
+        proj = rnd(n, 2 * H * D + 2 * H * Dv + 2 * H)
+        st, mx = torch.zeros(rows, H, Dv + 1, D, device=dev), torch.zeros(rows, H, Dv + 1, device=dev)
+        o, den = torch.empty(n, H * Dv, device=dev), torch.empty(n, H, device=dev)
+        hb, i_off = torch.zeros(H, device=dev), 2 * H * D + 2 * H * Dv
+        timed(f"mlstm_scan_{label}", lambda: K.mlstm_scan(proj, 0, H * D, 2 * H * D, i_off, i_off + H, hb, hb, 15.0,
+                                                          D ** -0.5, st, mx, cu, slots, o, den, rows),
+              nbytes=n * (2 * H * D + 2 * H * Dv + 3 * H) * 4 + rows * 2 * H * D * (Dv + 1) * 4)
+        gated, nw = torch.empty(n, H * Dv, dtype=bf, device=dev), torch.ones(H * Dv, device=dev)
+        timed(f"unit_norm_gate_{label}", lambda: K.unit_norm_gate(o, proj, 2 * H * D + H * Dv, gated, H, 1e-6, "sigmoid",
+                                                                  den=den, weight=nw), nbytes=n * H * Dv * 10)
+        q2, k2 = rnd(n, H, D), rnd(n, H, D)
+        st2, dec = torch.zeros(rows, H, Dv, D, device=dev), torch.full((H,), 0.97, device=dev)
+        timed(f"like:retention_scan_{label}", lambda: K.retention_scan(q2, k2, proj, 2 * H * D, dec, st2, cu, slots, o, rows),
+              nbytes=n * (2 * H * D + 2 * H * Dv) * 4 + rows * 2 * H * D * Dv * 4)
+        P_, N2 = 64, 128
+        C = width
+        u2, proj2 = rnd(n, C + 2 * N2), rnd(n, C // P_)
+        st3, y3, ones = torch.zeros(rows, C // P_, P_, N2, device=dev), torch.empty(n, C, device=dev), torch.ones(C // P_, device=dev)
+        timed(f"like:ssm_scan_{label}", lambda: K.ssm_scan(u2, proj2, 0, ones, ones, ones, st3, cu, slots, y3, rows,
+                                                          C // P_, P_, N2, 1),
+              nbytes=n * (2 * C + 2 * N2) * 4 + rows * 2 * C * N2 * 4)
+        # ---- the end of a layer -------------------------------------------------------------------------
+        h, y1, y2 = rnd(n, width), rnd(n, width), rnd(n, width)
+        xo = torch.empty(n, width, dtype=bf, device=dev)
+        timed(f"scaled_add_{label}", lambda: K.scaled_add(h, (y1, None, vec), (y2, None, vec), vec, 1e-6, xo),
+              nbytes=n * width * 18)
+        timed(f"like:norm_add_{label}", lambda: K.norm_add(h, y1, vec, 1e-6, 0.5, x_out=xo), nbytes=n * width * 14)
+        # ---- the router and the experts ---------------------------------------------------------------------
+        E, top, eff = 32, 4, ff // 4
+        logits = rnd(n, E + 1)
+        idx, wts = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+        timed(f"moe_route_groups_{label}", lambda: K.moe_route_groups(logits, idx, wts, top, E, 8, 5, 2.5))
+        timed(f"like:moe_route_scored_{label}", lambda: K.moe_route_scored(logits, None, idx, wts, top, E))
+        K.moe_route_groups(logits, idx, wts, top, E, 8, 5, 2.5)
+        wgu, wd = rnd(E, 2 * eff, width).to(bf), rnd(E, width, eff).to(bf)
+        if single:
+            pairs = wgu.view(E, eff, 2, width)
+            hid, hh = torch.empty(n, top, eff, dtype=bf, device=dev), torch.zeros(n, width, device=dev)
+            used = len(set(idx.flatten().tolist()))
+            timed("moe_experts_decode", lambda: K.moe_experts(x, pairs[:, :, 0], pairs[:, :, 1], wd, idx, wts, hid, hh,
+                                                              "clamped_swish", 7.0, 1.702, store=True),
+                  nbytes=used * 3 * width * eff * 2)
+        else:
+            np_ = n * top
+            counts, first = torch.zeros(E, dtype=torch.int32, device=dev), torch.empty(E + 1, dtype=torch.int32, device=dev)
+            order, where = torch.empty(np_, dtype=torch.int32, device=dev), torch.empty(n, top, dtype=torch.int32, device=dev)
+            K.moe_counts(idx, counts)
+            K.moe_place(idx, counts, first, order, where)
+            xg, act = torch.empty(np_, width, dtype=bf, device=dev), torch.empty(np_, eff, dtype=bf, device=dev)
+            K.moe_gather(x, order, xg, top)
+            yg = torch.empty(np_, width, device=dev)
+            timed("grouped_gate_up_prompt", lambda: K.gemm_tc_grouped(xg, wgu, act, first, status, "clamped_swish", 7.0, 1.702),
+                  flops=4.0 * np_ * width * eff)
+            timed("grouped_down_prompt", lambda: K.gemm_tc_grouped(act, wd, yg, first, status), flops=2.0 * np_ * width * eff)
+            at = first.tolist()
+
+            def one_by_one():
+                for e in range(E):
+                    if at[e + 1] > at[e]:
+                        K.gemm_tc_gated(xg[at[e]:at[e + 1]], wgu[e], act[at[e]:at[e + 1]], "clamped_swish", 7.0, 1.702, status)
+            timed("like:gate_up_an_expert_a_launch_prompt", one_by_one, flops=4.0 * np_ * width * eff)
+        # ---- latent attention ------------------------------------------------------------------------------------
+        kd, vd, rank, kw = 128, 128, PIKAVIK_RANK, PIKAVIK_RANK + 64
+        if not single:
+            qa, ka, va = (rnd(n, heads, 128).to(bf) for _ in range(3))
+            oa = torch.empty(n, heads * vd, dtype=bf, device=dev)
+            ctx = StepContext(device=torch.device(dev), act_dtype=bf, n_tokens=n, n_rows=1, token_ids=positions,
+                              positions=positions, token_row=token_row, cu_seqlens=cu, seq_end=cu[1:], slots=slots,
+                              from_start=True, single_token=False, max_row_tokens=n, max_end=n, status=status)
+            fl = heads * 2 * (kd + vd) * n * (n + 1) / 2
+            sink = rnd(heads)
+            for name, sl in (("latent_attention_prompt", sink), ("like:attention_prompt", None)):
+                spec = ScoreSpec(n_heads=heads, n_kv_heads=heads, head_dim=kd, value_dim=vd, scale=kd ** -0.5,
+                                 sink=sl is not None, sink_logit=sl)
+                timed(name, lambda: scored_attention(spec, qa, ka, va, None, ctx, oa), flops=fl)
+        else:
+            pages = tokens // 64 + 1
+            lat = rnd(rows * pages, 1, 64, kw).to(bf)
+            table = i32([[b * pages + p for p in range(pages)] for b in range(rows)])
+            pos1 = i32([tokens] * rows)
+            ql, ol = rnd(rows, heads, kw).to(bf), torch.empty(rows, heads * rank, dtype=bf, device=dev)
+            sink = rnd(heads)
+            timed("latent_decode", lambda: K.latent_decode(ql, lat, slots, pos1, table, pages, 0, ol, heads, kw, rank, 0, True,
+                                                           0.09, tokens + 1, sink_logit=sink), nbytes=rows * tokens * kw * 2)
+            kc, vc = rnd(rows * pages, heads // 4, 64, 128).to(bf), rnd(rows * pages, heads // 4, 64, 128).to(bf)
+            qd, od = rnd(rows, heads, 128).to(bf), torch.empty(rows, heads * 128, dtype=bf, device=dev)
+            cache = CacheView(k=kc, v=vc, page_table=table, table_stride=pages, ring=0)
+            ctx = StepContext(device=torch.device(dev), act_dtype=bf, n_tokens=rows, n_rows=rows, token_ids=pos1,
+                              positions=pos1, token_row=slots, cu_seqlens=cu, seq_end=i32([tokens + 1] * rows),
+                              slots=slots, from_start=False, single_token=True, max_row_tokens=1,
+                              max_end=tokens + 1, status=status)
+            spec = ScoreSpec(n_heads=heads, n_kv_heads=heads // 4, head_dim=128, value_dim=128, scale=128 ** -0.5,
+                             sink=True, sink_logit=sink)
+            timed("like:sink_attention_decode", lambda: scored_attention(spec, qd, None, None, cache, ctx, od),
+                  nbytes=rows * tokens * (heads // 4) * 2 * 128 * 2)
+            uk, uv = rnd(heads, rank, 64).to(bf), rnd(heads, 128, rank).to(bf)
+            qr, qa = rnd(rows, heads * 128).to(bf), torch.empty(rows, heads * kw, dtype=bf, device=dev)
+            timed("head_linear_queries_decode", lambda: K.head_linear(qr, uk, qa, x_head=128, x_off=0, y_head=kw, tail=64,
+                                                                      x_tail_off=64), nbytes=heads * rank * 64 * 2)
+            timed("head_linear_values_decode", lambda: K.head_linear(ol, uv, od.view(rows, -1), x_head=rank, x_off=0, y_head=128),
+                  nbytes=heads * rank * 128 * 2)
+    return out
+
+
+def workload_pikavik(args) -> int:
+    """Prefill of one 2,048-token prompt and decoding at batch 8 from 2,048-token contexts, for the
+    Pikavik design (WKV, mLSTM and latent-attention layers with routed feed-forwards) and for the Qwen2
+    decoder at equal width, feed-forward width a token and layers, random weights, bfloat16; and the
+    design's kernels alone."""
+    import torch
+    from minfer_b200.engine.generate import Generator
+    from minfer_b200.kernels import api as K
+    from minfer_b200.model import Model
+    pk, pk_kind = peaks()
+    torch.cuda.set_device(0)
+    steps = max(8, min(args.steps, 128))
+    clocks = ClockSampler()
+    clocks.start()
+    t_all = time.time()
+    sizes = []
+    for name, width, heads, ff, lstm_heads in PIKAVIK_SIZES:
+        cfg_p = pikavik_config(width, heads, ff, lstm_heads, FURITAR_VOCAB)
+        cfg_q = dict(CONFIG_7B, vocab_size=FURITAR_VOCAB, hidden_size=width, num_hidden_layers=PIKAVIK_LAYERS,
+                     num_attention_heads=heads, num_key_value_heads=heads // 4, intermediate_size=ff,
+                     max_position_embeddings=CONTEXT)
+        entry = {"name": name, "width": width, "heads": heads, "feed_forward": ff, "mlstm_heads": lstm_heads,
+                 "experts": 32, "experts_a_token": 4, "layers": PIKAVIK_LAYERS}
+        for label, cfg in (("pikavik", cfg_p), ("qwen2", cfg_q)):
+            model = Model.from_config(cfg, seed=0, dtype="bfloat16", device="cuda:0", make_on="device")
+            gen = Generator(model, max_tokens=BATCH * CONTEXT, max_batch=BATCH)
+            engine = gen.engine
+            g = torch.Generator().manual_seed(2)
+            ids = torch.randint(0, FURITAR_VOCAB, (PROMPT,), generator=g).tolist()
+            ms_prefill = time_prefill(engine, torch, ids, 10)
+            flops = pikavik_prefill_flops(cfg, PROMPT) if label == "pikavik" else prefill_flops(cfg, PROMPT)
+            ms_step, launched = time_decode(engine, torch, K, BATCH, steps, max(3, args.warmup), PROMPT)
+            ms_med = time_decode.median_ms
+            context = PROMPT + 3 + steps / 2
+            step_bytes = (pikavik_decode_bytes(model, cfg, BATCH, context) if label == "pikavik"
+                          else decode_bytes(model, BATCH, context))
+            entry[label] = {
+                "weights_gb": round(model.parameter_bytes() / 1e9, 3),
+                "prefill_tokens_per_s": round(PROMPT * 1e3 / ms_prefill, 1),
+                "prefill_ms": round(ms_prefill, 3),
+                "prefill_frac": round(flops / (ms_prefill * 1e-3) / (pk["bf16_tflops"] * 1e12), 4),
+                "decode_tokens_per_s": round(BATCH * 1e3 / ms_med, 1),
+                "decode_ms_per_step": round(ms_med, 4), "decode_frac": _frac(step_bytes, ms_med, pk),
+                "decode_launches_per_step": round(launched / steps, 1)}
+            del gen, engine, model
+            torch.cuda.empty_cache()
+        entry["kernels"] = pikavik_kernels(torch, K, pk, width, heads, ff, lstm_heads)
+        torch.cuda.empty_cache()
+        sizes.append(entry)
+    summary = clocks.summary((t_all, time.time()))
+    clocks.stop()
+    print(json.dumps({
+        "workload": "pikavik", "impl": "ours", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
+        "metric": "prefill tokens/s of one 2048-token prompt and decode tokens/s at batch 8 from "
+                  "2048-token contexts, Pikavik beside Qwen2 at equal width and layers",
+        "unit": "tokens/s", "steps": steps, "prompt_len": PROMPT, "batch": BATCH,
+        "fractions": f"prefill: flops over the {pk_kind} bf16 product peak; decode: bytes of the "
+                     f"weights a step touches, the latent vectors of the context and the recurrent "
+                     f"state over the {pk_kind} copy bandwidth",
+        "l2": "weights larger than L2 are read every step; kernels alone: L2 flushed before each run",
+        "clocks": summary, "sizes": sizes}))
+    return 0
+
+
 REF_KERNELS = os.path.join(ROOT, "baseline", "_ref", "libref_kernels.so")
 # the reference's checkout, if it sits beside this repository (or where MINFER_REFERENCE_DIR says)
 REF_SOURCE = os.path.join(os.environ.get("MINFER_REFERENCE_DIR",
@@ -1457,7 +1748,7 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=None,
                     help="run fewer layers than the configuration has (both numbers are reported)")
-    ap.add_argument("--workload", default="qwen2-7b", choices=["qwen2-7b", "furitar", "budanex", "bedarax", "zanelorn"],
+    ap.add_argument("--workload", default="qwen2-7b", choices=["qwen2-7b", "furitar", "budanex", "bedarax", "zanelorn", "pikavik"],
                     help="qwen2-7b (the default): the headline figure and its points; furitar: "
                          "the Furitar design beside Qwen2 at equal sizes, prefill and decode")
     ap.add_argument("--skip-points", action="store_true",
@@ -1482,6 +1773,8 @@ def main() -> int:
         return workload_bedarax(args)
     if args.workload == "zanelorn":
         return workload_zanelorn(args)
+    if args.workload == "pikavik":
+        return workload_pikavik(args)
 
     import torch
     from minfer_b200.engine.generate import Generator

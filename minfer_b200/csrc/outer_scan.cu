@@ -139,7 +139,10 @@ __global__ void __launch_bounds__(OS_THREADS) outer_scan_kernel(OuterScanArgs a,
     const bool live0 = 2 * c < n_cols, live1 = 2 * c + 1 < n_cols;
     const int t0 = a.cu_seqlens[b], n_b = a.cu_seqlens[b + 1] - t0;
     const int slot = a.slots[b];
-    const bool vec = (D & 3) == 0 && ((a.r_width | a.k_width | a.w_width | (long long)(a.r_off | a.k_off | a.w_off)) & 3) == 0;
+    // (a row of a tensor may start anywhere: 16-byte copies only where all of them start on 16 bytes)
+    const bool vec = (D & 3) == 0 &&
+                     ((a.r_width | a.k_width | a.w_width | (long long)(a.r_off | a.k_off | a.w_off)) & 3) == 0 &&
+                     (((uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.w) & 15) == 0;
     if (DP > D) {                                      // the copies never touch the padding
         const int pad = DP - D;
         for (int i = tid; i < 2 * tc * NVEC * pad; i += OS_THREADS) {
@@ -262,7 +265,9 @@ __global__ void __launch_bounds__(OS_THREADS) outer_scan_kernel(OuterScanArgs a,
             float before = __shfl_up_sync(0xffffffffu, m_t, 1);
             if (lane == 0) before = m_run;
             if (mine) {
-                keep_s[lane] = expf(lf + before - m_t);
+                // (m_t is often lf + before, rounded: in this order the difference is exact, so what m_t lost
+                // in rounding stays in the state's factor instead of adding up token by token)
+                keep_s[lane] = expf((before - m_t) + lf);
                 add_s[lane] = expf(li - m_t);
                 floor_s[lane] = expf(-m_t);
             }
@@ -364,8 +369,7 @@ template <bool WKV>
 static int os_choose(const OuterScanArgs& a, cudaStream_t stream) {
     if (a.n_rows <= 0) return 0;
     if (a.D < 1 || a.D > OS_MAX_D || a.Dv < 1 || a.heads < 1 || a.n_rows > 65535) return MF_ERR_UNSUPPORTED;
-    const uintptr_t ptrs = (uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.w | (uintptr_t)a.state;
-    if ((ptrs & 15) != 0) return MF_ERR_UNSUPPORTED;
+    if (((uintptr_t)a.state & 15) != 0) return MF_ERR_UNSUPPORTED;
     if (a.D <= 32) return os_launch<8, 1, WKV>(a, stream);
     if (a.D <= 64) return os_launch<16, 1, WKV>(a, stream);
     if (a.D <= 128) return os_launch<16, 2, WKV>(a, stream);

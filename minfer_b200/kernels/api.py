@@ -167,6 +167,13 @@ def _sig_attention_sink(lib: ctypes.CDLL) -> None:
                                                             c_void_p])
 
 
+def _sig_attention_latent(lib: ctypes.CDLL) -> None:
+    lib.mf_latent_supported.argtypes = [c_int, c_int]
+    lib.mf_latent_plan.argtypes = [c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+    lib.mf_latent_decode.argtypes = ([c_void_p] * 5 + [c_int, c_int, c_void_p, c_void_p] + [c_int] * 6 +
+                                     [c_float, c_int, c_void_p, c_void_p])
+
+
 def _sig_sampling(lib: ctypes.CDLL) -> None:
     lib.mf_sample.argtypes = [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p,
                               c_void_p, c_float, c_int, c_float, c_float, c_float, c_float,
@@ -289,7 +296,7 @@ def _sig_moe(lib: ctypes.CDLL) -> None:
 _SIGNATURES = {"retention": _sig_retention, "outer_scan": _sig_outer_scan, "delta_rule": _sig_delta_rule, "attention_talk": _sig_attention_talk, "moe": _sig_moe,
                "attention_prefill_tc": _sig_attention_prefill_tc, "recurrent": _sig_recurrent,
                "mixer_prep": _sig_mixer_prep,
-               "attention_sink": _sig_attention_sink,
+               "attention_sink": _sig_attention_sink, "attention_latent": _sig_attention_latent,
                "attention_prefill": _sig_attention_prefill, "gemm_tc": _sig_gemm_tc, "ops": _sig_ops, "gemm_simt": _sig_gemm_simt, "attention": _sig_attention,
                "sampling": _sig_sampling}
 
@@ -1937,6 +1944,41 @@ def sink_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
         n_kv, head_dim, value_dim, int(window), int(chunk), 1 if sink else 0, float(scale),
         int(reach_keys), _f32(sink_logit, "sink_logit"), float(softcap), int(keep_first), _stream()),
         "sink_attention_decode", 2 if splits > 1 else 1)
+
+
+def latent_decode_supported(dtype: torch.dtype, key_dim: int, value_dim: int) -> bool:
+    """The kernel over wide latent vectors takes bfloat16, vectors of up to 640 numbers of which the
+    first ``value_dim`` are the value, both multiples of 8."""
+    return (dtype == torch.bfloat16 and 8 <= value_dim <= key_dim <= 640 and key_dim % 8 == 0
+            and value_dim % 8 == 0)
+
+
+def latent_decode(q: torch.Tensor, cache: torch.Tensor, row_seq: torch.Tensor, row_pos: torch.Tensor,
+                  page_table: torch.Tensor, table_stride: int, ring: int, out: torch.Tensor, n_heads: int,
+                  key_dim: int, value_dim: int, window: int, sink: bool, scale: float, reach_keys: int,
+                  sink_logit: Optional[torch.Tensor] = None) -> None:
+    """Every row of ``q`` [rows, heads, key_dim] is a query at its own position over the paged cache of
+    latent vectors (one key/value head): out [rows, heads * value_dim] = softmax-weighted sums of the
+    vectors' first ``value_dim`` numbers.  ``reach_keys``: the most keys a query sees."""
+    rows = q.shape[0]
+    if (q.dtype != torch.bfloat16 or q.numel() != rows * n_heads * key_dim or cache.shape[-1] != key_dim
+            or cache.shape[1] != 1 or out.shape != (rows, n_heads * value_dim)):
+        raise KernelError("latent_decode: bfloat16 only, shapes must fit")
+    lib = _lib("attention_latent")
+    key = ("latent", rows, n_heads, key_dim, int(reach_keys))
+    splits = _SINK_PLANS.get(key)
+    if splits is None:
+        tpc, sp = ctypes.c_int(0), ctypes.c_int(0)
+        lib.mf_latent_plan(rows, n_heads, key_dim, int(reach_keys), ctypes.addressof(tpc), ctypes.addressof(sp))
+        splits = _SINK_PLANS[key] = sp.value
+    partial = None
+    if splits > 1:
+        partial = torch.empty(rows * n_heads * splits * (value_dim + 2), dtype=torch.float32, device=q.device)
+    _check(lib.mf_latent_decode(
+        _ptr(q, "q"), _ptr(cache, "cache"), _i32(row_seq, "row_seq"), _i32(row_pos, "row_pos"),
+        _i32(page_table, "page_table"), int(table_stride), int(ring), _ptr(out, "out"), _f32(partial, "partial"),
+        rows, n_heads, key_dim, value_dim, int(window), 1 if sink else 0, float(scale), int(reach_keys),
+        _f32(sink_logit, "sink_logit"), _stream()), "latent_decode", 2 if splits > 1 else 1)
 
 
 def sampler_state_ints() -> int:

@@ -56,6 +56,8 @@ class LatentAttention(Mixer):
     def libraries(self, dtype: torch.dtype) -> List[str]:
         libs = ["ops", "mixer_prep", "attention_sink"]
         libs.append("gemm_tc" if dtype == torch.bfloat16 else "gemm_simt")
+        if self._wide(dtype):
+            libs.append("attention_latent")
         kw = self.kv_rank + self.rot_dim
         if (K.sink_attention_tc_supported(dtype, kw, kw)
                 or K.sink_attention_tc_supported(dtype, self.head_dim + self.rot_dim, self.value_dim)):
@@ -170,10 +172,17 @@ class LatentAttention(Mixer):
                          scale=self.scale, window=self.window, sink=self.sink,
                          sink_logit=self.sink_logit)
 
+    def _wide(self, act: torch.dtype) -> bool:
+        """The kernel for wide latent vectors runs this part's absorbed form."""
+        kw = self.kv_rank + self.rot_dim
+        return (K.latent_decode_supported(act, kw, self.kv_rank)
+                and not K.sink_attention_mma_supported(act, kw, kw))
+
     def _expanded_scores(self) -> Optional[ScoreSpec]:
         """The attention over expanded keys and values, where the kernels for prompts take its sizes."""
         kd, vd = self.head_dim + self.rot_dim, self.value_dim
-        if (not EXPAND_PROMPTS or self.uv.dtype != torch.bfloat16 or self.kv_rank % 8 or self.rot_dim % 8
+        if (not EXPAND_PROMPTS or self._uk.dtype != torch.bfloat16 or self._uv.dtype != torch.bfloat16
+                or self.kv_rank % 8 or self.rot_dim % 8
                 or not K.sink_attention_mma_supported(torch.bfloat16, kd, vd)):
             return None
         return ScoreSpec(n_heads=self.n_heads, n_kv_heads=self.n_heads, head_dim=kd, value_dim=vd,
@@ -242,11 +251,13 @@ class LatentAttention(Mixer):
                          v_off=0, v_width=rank, v_from_k=True, q_norm=None, k_norm=None,
                          eps=self.norm_eps, inv_freq=inv_freq, rot_dims=rot_dims, rot_style=style,
                          rot_magnitude=magnitude, q_rot_off=hd, k_rot_off=rank, status=ctx.status)
-        expanded = self._expanded_scores() if own_kv and act == torch.bfloat16 and not self.gate else None
+        expanded = self._expanded_scores() if own_kv and act == torch.bfloat16 else None
         if expanded is not None:
             k_all, v_all = self._expand(k_step.view(n, kw))
             o = torch.empty((n, nh * vd), dtype=act, device=dev)
             scored_attention(expanded, q.view(n, nh, hd + rd), k_all, v_all, cache, ctx, o)
+            if self.gate:
+                K.gate_mul(o, proj, nq + kw)
             project_out(self.out, o, ctx, residual)
             return
         if self.uk_t.dtype != act:
@@ -256,10 +267,20 @@ class LatentAttention(Mixer):
         # q'_h = [Wuk_h^T q_p | q_r]
         q_abs = torch.empty((n, nh * kw), dtype=act, device=dev)
         K.head_linear(q, self.uk_t, q_abs, x_head=hd + rd, x_off=0, y_head=kw, tail=rd, x_tail_off=hd)
-        o_lat = torch.empty((n, nh * kw), dtype=act, device=dev)
-        scored_attention(self.scores(), q_abs.view(n, nh, kw), k_step, k_step, cache, ctx, o_lat)
+        # vectors wider than the other kernels take: every token a query over the cache's pages, which
+        # hold the step's vectors by now (unless a ring has dropped some that a prompt's tokens see)
+        wide = (self._wide(act) and not (own_kv and cache.ring))
+        v_head = rank if wide else kw
+        o_lat = torch.empty((n, nh * v_head), dtype=act, device=dev)
+        if wide:
+            reach = self.window if self.window > 0 else ctx.max_end
+            K.latent_decode(q_abs.view(n, nh, kw), cache.k, ctx.token_row, ctx.positions, cache.page_table,
+                            cache.table_stride, cache.ring, o_lat, nh, kw, rank, self.window, self.sink,
+                            self.scale, reach, sink_logit=self.sink_logit)
+        else:
+            scored_attention(self.scores(), q_abs.view(n, nh, kw), k_step, k_step, cache, ctx, o_lat)
         # o_h = Wuv_h (the first kv_rank columns of the weighted sum), times the gate
         o = torch.empty((n, nh * vd), dtype=act, device=dev)
-        K.head_linear(o_lat, self.uv, o, x_head=kw, x_off=0, y_head=vd,
+        K.head_linear(o_lat, self.uv, o, x_head=v_head, x_off=0, y_head=vd,
                       gate=proj if self.gate else None, gate_off=nq + kw)
         project_out(self.out, o, ctx, residual)

@@ -173,28 +173,32 @@ def clamped_expert(x: torch.Tensor, w: Mapping[str, torch.Tensor], p: str, limit
     return (g * torch.sigmoid(1.702 * g) * (u + 1.0)) @ w[p + "down"].T
 
 
-def choose(s: torch.Tensor, top: int, groups: int, keep: int, scale: float):
-    """From scores [T, experts]: (chosen [T, top], weights [T, top], margin [T]): the margin is how
-    far, as a fraction of the scores concerned, the closest of the two choices (groups, experts) was."""
+def choose(z: torch.Tensor, top: int, groups: int, keep: int, scale: float):
+    """From router outputs z [T, experts]: (chosen [T, top], weights [T, top], margin [T]).  The margin
+    says how far the closest of the two choices (groups, experts) was: the relative change of a token's
+    z that it takes, to first order, to turn it."""
+    s = torch.sigmoid(z)
     T, E = s.shape
-    inf = torch.full((T,), float("inf"), dtype=s.dtype)
-    margin = inf
+    # what s moves by when every z moves by its typical size
+    moves = s * (1.0 - s) * (z * z).mean(dim=-1, keepdim=True).sqrt().clamp(min=0.1)
+    margin = torch.full((T,), float("inf"), dtype=s.dtype)
     allowed = torch.ones(T, E, dtype=torch.bool)
     if groups > 1 and keep < groups:
         size = E // groups
-        best = torch.sort(s.view(T, groups, size), dim=-1, descending=True).values[..., :2].sum(-1)
+        two = torch.topk(s.view(T, groups, size), min(2, size), dim=-1)
+        best = two.values.sum(-1)
+        give = torch.gather(moves.view(T, groups, size), 2, two.indices).sum(-1)
         order = torch.argsort(best, dim=-1, descending=True, stable=True)
-        ranked = torch.gather(best, 1, order)
-        margin = torch.minimum(margin, (ranked[:, keep - 1] - ranked[:, keep])
-                               / ranked[:, keep - 1].clamp(min=1e-30))
+        ranked, give = torch.gather(best, 1, order), torch.gather(give, 1, order)
+        margin = (ranked[:, keep - 1] - ranked[:, keep]) / (give[:, keep - 1] + give[:, keep]).clamp(min=1e-30)
         ok = torch.zeros(T, groups, dtype=torch.bool).scatter_(1, order[:, :keep], True)
         allowed = ok.repeat_interleave(size, dim=1)
     masked = s.masked_fill(~allowed, float("-inf"))
     order = torch.argsort(masked, dim=-1, descending=True, stable=True)
-    ranked = torch.gather(masked, 1, order)
-    if top < E:
+    ranked, give = torch.gather(masked, 1, order), torch.gather(moves, 1, order)
+    if top < int(allowed[0].sum()):
         margin = torch.minimum(margin, (ranked[:, top - 1] - ranked[:, top])
-                               / ranked[:, top - 1].clamp(min=1e-30))
+                               / (give[:, top - 1] + give[:, top]).clamp(min=1e-30))
     chosen = order[:, :top]
     picked = torch.gather(s, 1, chosen)
     return chosen, picked / (picked.sum(-1, keepdim=True) + 1e-20) * scale, margin
@@ -204,8 +208,7 @@ def routed_ff(y: torch.Tensor, w: Mapping[str, torch.Tensor], p: str, mlp: Mappi
               margins: Optional[List[torch.Tensor]] = None) -> torch.Tensor:
     r = mlp["router"]
     g = r.get("groups") or {"count": 1, "keep": 1}
-    s = torch.sigmoid(y @ w[p + "router"].T)
-    chosen, weight, margin = choose(s, r["top"], g["count"], g["keep"], r.get("scale", 1.0))
+    chosen, weight, margin = choose(y @ w[p + "router"].T, r["top"], g["count"], g["keep"], r.get("scale", 1.0))
     if margins is not None:
         margins.append(margin)
     out = torch.zeros_like(y)
