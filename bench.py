@@ -1422,7 +1422,7 @@ def pikavik_kernels(torch, K, pk, width, heads, ff, lstm_heads, tokens=2048, bat
         timed(f"wkv_decay_{label}", lambda: K.wkv_decay(t1, w2t, w0, decay), nbytes=n * (64 + H * D) * 4 + 64 * H * D * 4)
         r, k, v, u = rnd(n, H * D), rnd(n, H * D) * 0.1, rnd(n, H * D), rnd(H, D)
         state, o = torch.zeros(rows, H, D, D, device=dev), torch.empty(n, H * D, device=dev)
-        timed(f"wkv_scan_{label}", lambda: K.wkv_scan(r, k, v, decay, u, state, cu, slots, o, rows),
+        timed(f"wkv_scan_{label}", lambda: K.wkv_scan(r, k, v, decay, u, state, cu, slots, o, rows, per),
               nbytes=n * 5 * H * D * 4 + rows * 2 * H * D * D * 4)
         # ---- mLSTM beside retention of the same keys and values ---------------------------------------------
         H, D, Dv = lstm_heads, 128, 256
@@ -1431,7 +1431,7 @@ def pikavik_kernels(torch, K, pk, width, heads, ff, lstm_heads, tokens=2048, bat
         o, den = torch.empty(n, H * Dv, device=dev), torch.empty(n, H, device=dev)
         hb, i_off = torch.zeros(H, device=dev), 2 * H * D + 2 * H * Dv
         timed(f"mlstm_scan_{label}", lambda: K.mlstm_scan(proj, 0, H * D, 2 * H * D, i_off, i_off + H, hb, hb, 15.0,
-                                                          D ** -0.5, st, mx, cu, slots, o, den, rows),
+                                                          D ** -0.5, st, mx, cu, slots, o, den, rows, per),
               nbytes=n * (2 * H * D + 2 * H * Dv + 3 * H) * 4 + rows * 2 * H * D * (Dv + 1) * 4)
         gated, nw = torch.empty(n, H * Dv, dtype=bf, device=dev), torch.ones(H * Dv, device=dev)
         timed(f"unit_norm_gate_{label}", lambda: K.unit_norm_gate(o, proj, 2 * H * D + H * Dv, gated, H, 1e-6, "sigmoid",
@@ -1468,6 +1468,17 @@ def pikavik_kernels(torch, K, pk, width, heads, ff, lstm_heads, tokens=2048, bat
             timed("moe_experts_decode", lambda: K.moe_experts(x, pairs[:, :, 0], pairs[:, :, 1], wd, idx, wts, hid, hh,
                                                               "clamped_swish", 7.0, 1.702, store=True),
                   nbytes=used * 3 * width * eff * 2)
+            first = torch.empty(E + 1, dtype=torch.int32, device=dev)
+            where = torch.empty(n, top, dtype=torch.int32, device=dev)
+            xg, act = torch.empty(n * top, width, dtype=bf, device=dev), torch.empty(n * top, eff, dtype=bf, device=dev)
+            yg = torch.empty(n * top, width, device=dev)
+
+            def grouped():
+                K.moe_group_few(idx, x, E, xg, first, where)
+                K.gemm_tc_grouped(xg, wgu, act, first, status, "clamped_swish", 7.0, 1.702)
+                K.gemm_tc_grouped(act, wd, yg, first, status)
+                K.moe_combine(yg, where, wts, hh, store=True)
+            timed("moe_grouped_decode", grouped, nbytes=used * 3 * width * eff * 2)
         else:
             np_ = n * top
             counts, first = torch.zeros(E, dtype=torch.int32, device=dev), torch.empty(E + 1, dtype=torch.int32, device=dev)

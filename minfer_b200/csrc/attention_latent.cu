@@ -233,28 +233,35 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_decode_kernel(LatentArgs
     }
 }
 
-// merges the splits of one (query, head) in split order and adds the sink
-__global__ void __launch_bounds__(128)
+// Merges the splits of one (query, head) in split order and adds the sink.  The splits' factors are
+// formed once, then every output number is a sum of independent loads.
+#define LA_MAX_SPLITS 512
+__global__ void __launch_bounds__(256)
 latent_combine_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ out, int n_splits, int vd,
                       int sink, const float* __restrict__ sink_logit, int n_heads) {
     pdl_prologue();
+    __shared__ float f_s[LA_MAX_SPLITS];
+    __shared__ float scratch[33];
     const size_t rh = blockIdx.x, stride = (size_t)(vd + 2);
     const float* p = partial + rh * n_splits * stride;
     const float sink2 = (sink && sink_logit) ? sink_logit[rh % n_heads] * 1.4426950408889634f : 0.f;
     float m = sink ? sink2 : -INFINITY;
-    for (int c = 0; c < n_splits; ++c) m = fmaxf(m, p[c * stride]);
-    float l = sink ? exp2f(sink2 - m) : 0.f;
-    for (int c = 0; c < n_splits; ++c) {
-        const float mc = p[c * stride];
-        if (mc > -INFINITY) l = fmaf(p[c * stride + 1], exp2f(mc - m), l);
+    for (int c = threadIdx.x; c < n_splits; c += blockDim.x) m = fmaxf(m, p[c * stride]);
+    m = block_max(m, scratch);
+    float l = 0.f;
+    for (int c = threadIdx.x; c < n_splits; c += blockDim.x) {
+        const float f = exp2f(p[c * stride] - m);      // (a split that saw nothing has maximum -inf: 0)
+        f_s[c] = f;
+        l = fmaf(p[c * stride + 1], f, l);
     }
+    l = block_sum(l, scratch);                         // (its barriers also publish f_s)
+    if (sink) l += exp2f(sink2 - m);
     const float inv = 1.0f / l;
     for (int d = threadIdx.x; d < vd; d += blockDim.x) {
+        const float* pd = p + 2 + d;
         float acc = 0.f;
-        for (int c = 0; c < n_splits; ++c) {
-            const float mc = p[c * stride];
-            if (mc > -INFINITY) acc = fmaf(p[c * stride + 2 + d], exp2f(mc - m), acc);
-        }
+#pragma unroll 8
+        for (int c = 0; c < n_splits; ++c) acc = fmaf(pd[c * stride], f_s[c], acc);
         out[rh * vd + d] = __float2bfloat16_rn(acc * inv);
     }
 }
@@ -273,6 +280,7 @@ extern "C" int mf_latent_plan(int rows, int n_heads, int kw, int reach_keys, int
     if (per_sm < 1) per_sm = 1;
     int splits = blocks > 0 ? (per_sm * mf_sm_count()) / blocks : 1;
     if (splits > n_tiles) splits = n_tiles;
+    if (splits > LA_MAX_SPLITS) splits = LA_MAX_SPLITS;
     if (splits < 1) splits = 1;
     const int tpc = (n_tiles + splits - 1) / splits;
     *tiles_per_cta = tpc;
@@ -324,7 +332,7 @@ extern "C" int mf_latent_decode(const void* q, const void* k_cache, const int* r
     else if (vd <= 512) e = la_launch<4>(a, rows, stream);
     else e = la_launch<5>(a, rows, stream);
     if (e || a.n_splits == 1) return e;
-    mf_launch_ex(false, latent_combine_kernel, dim3(rows * n_heads), dim3(128), 0, stream, (const float*)partial,
+    mf_launch_ex(false, latent_combine_kernel, dim3(rows * n_heads), dim3(vd <= 128 ? 128 : 256), 0, stream, (const float*)partial,
                  (__nv_bfloat16*)out, a.n_splits, vd, a.sink, sink_logit, n_heads);
     return MF_LAUNCH_CHECK();
 }

@@ -539,6 +539,57 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(HeadLinearArgs a) 
     }
 }
 
+// Few tokens (bfloat16): a warp per (head, output), which reads its row of W once, 16 bytes a lane at a
+// time, and forms the sums of up to HF_T tokens side by side; the tokens' inputs come from L1.
+#define HF_T 8
+__global__ void __launch_bounds__(256) head_linear_few_kernel(HeadLinearArgs a) {
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const int out = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int h = blockIdx.y, t0 = blockIdx.z * HF_T, nt = min(HF_T, a.n_tokens - t0);
+    const __nv_bfloat16* x = (const __nv_bfloat16*)a.x + (size_t)t0 * a.x_row + (size_t)h * a.x_head + a.x_off;
+    __nv_bfloat16* y = (__nv_bfloat16*)a.y + (size_t)t0 * a.y_row + (size_t)h * a.y_head;
+    const bool live = out < a.J;
+    const __nv_bfloat16* w = (const __nv_bfloat16*)a.w + ((size_t)h * a.J + (live ? out : 0)) * a.D;
+    pdl_wait();
+    if (a.tail > 0 && blockIdx.x == 0)
+        for (int i = threadIdx.x; i < nt * a.tail; i += blockDim.x) {
+            const int t = i / a.tail, c = i - t * a.tail;
+            y[(size_t)t * a.y_row + a.J + c] = ((const __nv_bfloat16*)a.x)[(size_t)(t0 + t) * a.x_row + (size_t)h * a.x_head + a.x_tail_off + c];
+        }
+    if (!live) return;
+    float acc[HF_T];
+#pragma unroll
+    for (int t = 0; t < HF_T; ++t) acc[t] = 0.f;
+    for (int d = lane * 8; d < a.D; d += 256) {
+        const uint4 wv = *reinterpret_cast<const uint4*>(w + d);
+        const unsigned wu[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+        for (int t = 0; t < HF_T; ++t) {
+            if (t >= nt) break;
+            const uint4 xv = *reinterpret_cast<const uint4*>(x + (size_t)t * a.x_row + d);
+            const unsigned xu[4] = {xv.x, xv.y, xv.z, xv.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                acc[t] = fmaf(__uint_as_float(wu[e] << 16), __uint_as_float(xu[e] << 16), acc[t]);
+                acc[t] = fmaf(__uint_as_float(wu[e] & 0xffff0000u), __uint_as_float(xu[e] & 0xffff0000u), acc[t]);
+            }
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < HF_T; ++t) {
+        if (t >= nt) break;
+        float v = warp_sum(acc[t]);
+        if (lane == 0) {
+            if (a.gate != nullptr) {
+                const float g = a.gate[(size_t)(t0 + t) * a.gate_row + a.gate_off + (size_t)h * a.J + out];
+                v *= 1.0f / (1.0f + expf(-g));
+            }
+            y[(size_t)t * a.y_row + out] = __float2bfloat16_rn(v);
+        }
+    }
+}
+
 extern "C" int mf_head_linear(const HeadLinearArgs* args, int dtype, cudaStream_t stream) {
     const HeadLinearArgs a = *args;
     if (a.n_tokens <= 0) return 0;
@@ -546,6 +597,12 @@ extern "C" int mf_head_linear(const HeadLinearArgs* args, int dtype, cudaStream_
     dim3 grid((a.n_tokens + HL_TT - 1) / HL_TT, (a.J + HL_TJ - 1) / HL_TJ, a.heads);
     static int simt = -1;              // MINFER_B200_HEAD_LINEAR=simt: the FP32-pipe kernel for bfloat16 too
     if (simt < 0) { const char* e = getenv("MINFER_B200_HEAD_LINEAR"); simt = (e && e[0] == 's') ? 1 : 0; }
+    if (dtype == MF_DTYPE_BF16 && !simt && a.n_tokens <= 16 && a.heads <= 65535 &&
+        ((a.D | a.x_head | a.x_off) & 7) == 0 && (a.x_row & 7) == 0 && (((uintptr_t)a.x | (uintptr_t)a.w) & 15) == 0) {
+        mf_launch(head_linear_few_kernel, dim3((a.J + 7) / 8, a.heads, (a.n_tokens + HF_T - 1) / HF_T), dim3(256), 0,
+                  stream, a);
+        return MF_LAUNCH_CHECK();
+    }
     if (dtype == MF_DTYPE_F32) mf_launch(head_linear_kernel<float>, grid, dim3(256), 0, stream, a);
     else if (dtype == MF_DTYPE_BF16 && !simt) mf_launch(head_linear_mma_kernel, grid, dim3(128), 0, stream, a);
     else if (dtype == MF_DTYPE_BF16) mf_launch(head_linear_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, a);

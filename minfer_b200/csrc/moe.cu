@@ -469,10 +469,64 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict
     for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = xr[i];
 }
 
+// the same 16 bytes a thread at a time, for rows that are whole numbers of them
+__global__ void __launch_bounds__(256)
+moe_gather_vec_kernel(const uint4* __restrict__ x, const int* __restrict__ pairs, uint4* __restrict__ out,
+                      int per_row, int top) {
+    pdl_prologue();
+    const uint4* xr = x + (size_t)(pairs[blockIdx.x] / top) * per_row;
+    uint4* o = out + (size_t)blockIdx.x * per_row;
+    for (int i = threadIdx.x; i < per_row; i += blockDim.x) o[i] = xr[i];
+}
+
+// moe_counts, moe_place and moe_gather in one launch, for steps of few pairs: a block per pair counts
+// the pairs before it (experts in order, an expert's pairs in their order), which is its row, and
+// copies the token's input there; the first block also writes the experts' first rows.
+__global__ void __launch_bounds__(256)
+moe_group_few_kernel(const int* __restrict__ idx, int n_pairs, int experts, int top, const uint4* __restrict__ x,
+                     uint4* __restrict__ out, int per_row, int* __restrict__ offsets, int* __restrict__ where) {
+    pdl_prologue();
+    extern __shared__ int mg_idx[];
+    __shared__ int mg_pos;
+    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) mg_idx[i] = idx[i];
+    if (threadIdx.x == 0) mg_pos = 0;
+    __syncthreads();
+    const int p = blockIdx.x, e = mg_idx[p];
+    int before = 0;
+    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) before += (mg_idx[i] < e) || (mg_idx[i] == e && i < p);
+    if (before) atomicAdd(&mg_pos, before);
+    __syncthreads();
+    const int pos = mg_pos;
+    if (threadIdx.x == 0) where[p] = pos;
+    const uint4* xr = x + (size_t)(p / top) * per_row;
+    uint4* o = out + (size_t)pos * per_row;
+    for (int i = threadIdx.x; i < per_row; i += blockDim.x) o[i] = xr[i];
+    if (p == 0)
+        for (int g = threadIdx.x; g <= experts; g += blockDim.x) {
+            int below = 0;
+            for (int i = 0; i < n_pairs; ++i) below += mg_idx[i] < g;
+            offsets[g] = below;
+        }
+}
+
+extern "C" int mf_moe_group_few(const int* idx, int n_pairs, int experts, int top, const void* x, void* out,
+                                int row_bytes, int* offsets, int* where, cudaStream_t stream) {
+    if (n_pairs <= 0) return 0;
+    if (n_pairs > 4096 || experts < 1 || top < 1 || row_bytes % 16 != 0 || (((uintptr_t)x | (uintptr_t)out) & 15))
+        return MF_ERR_UNSUPPORTED;
+    mf_launch(moe_group_few_kernel, dim3(n_pairs), dim3(256), (size_t)n_pairs * sizeof(int), stream, idx, n_pairs,
+              experts, top, (const uint4*)x, (uint4*)out, row_bytes / 16, offsets, where);
+    return MF_LAUNCH_CHECK();
+}
+
 extern "C" int mf_moe_gather(const void* x, int dtype, const int* pairs, void* out, int n, int width,
                              int top, cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (dtype == MF_DTYPE_F32)
+    const size_t bytes = (size_t)width * (dtype == MF_DTYPE_F32 ? 4 : 2);
+    if ((dtype == MF_DTYPE_F32 || dtype == MF_DTYPE_BF16) && bytes % 16 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0)
+        mf_launch(moe_gather_vec_kernel, dim3(n), dim3(bytes / 16 >= 256 ? 256 : 128), 0, stream, (const uint4*)x, pairs,
+                  (uint4*)out, (int)(bytes / 16), top);
+    else if (dtype == MF_DTYPE_F32)
         mf_launch(moe_gather_kernel<float>, dim3(n), dim3(256), 0, stream, (const float*)x, pairs,
                   (float*)out, width, top);
     else if (dtype == MF_DTYPE_BF16)

@@ -11,20 +11,23 @@
 //                 one more column of S, whose value is always 1.
 //   wkv_decay     w = exp(-exp(w0 + W2 tanh(t1))) per token and channel, W2 through a small rank
 //
-// The scan: a block owns (row, head, a tile of columns); LD neighbouring lanes share a pair of
-// columns and hold its state elements d = 4 (l + LD i) .. + 3 in registers, so that what a lane
-// reads of q, k and the decays from shared memory (16 bytes at a time) serves two columns.  Tokens
-// come in chunks through two cp.async buffers, four tokens' sums side by side: their eight numbers
-// are summed over the lanes by halving (each step sends what the partner keeps), 4 + 2 + 1
-// shuffles and one more for every doubling of LD beyond 8.  A sum's tree does not depend on the
-// chunk, so the cut of a sequence changes nothing but the order of nothing.
+// The scan: a block owns (row, head, a tile of columns).  Four warps walk the tokens: LD neighbouring
+// lanes share a pair of columns and hold its state elements d = 4 (l + LD i) .. + 3 in registers, so
+// that what a lane reads of q, k and the decays from shared memory (16 bytes at a time) serves two
+// columns.  The sums of eight tokens (16 numbers a lane) are formed side by side and added over the
+// lanes by halving: each step sends what the partner keeps, 8 + 4 + 2 + 1 shuffles for all of them.  A
+// sum's tree does not depend on how the tokens are grouped.  A fifth warp does what is not the chain:
+// it keeps a ring of three chunks of tokens filled by cp.async and prepares each (wkv: r . (u k); mlstm:
+// gates and maxima), handing chunks over and taking them back through named barriers.
 // State [slots][heads][columns][D]: a column's elements are contiguous.  Every column keeps its own
 // copy of the running maximum ([slots][heads][columns]), so no block reads what another writes.
 // Tokens are packed row after row (row b: tokens cu_seqlens[b] .. cu_seqlens[b + 1]).
 #include "common.cuh"
 
-#define OS_THREADS 128
-#define OS_TU 4              // tokens whose sums are formed side by side
+#define OS_THREADS 128       // the threads that walk the tokens; one more warp feeds them
+#define OS_TU 8              // tokens whose sums are formed side by side
+#define OS_TC 16             // tokens of a chunk
+#define OS_STAGES 3
 #define OS_MAX_D 256
 
 struct OuterScanArgs {
@@ -57,13 +60,14 @@ __device__ __forceinline__ void os_cp16(float* dst, const float* src) {
                  ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// Sums the 8 numbers of every lane over groups of LD lanes.  The lane with index l of its group gets
-// number l / (LD / 8), complete.
+// Sums the 16 numbers of every lane over groups of LD lanes.  The lane with index l of its group gets
+// LD 8: numbers 2 l and 2 l + 1 (in a[0], a[1]); LD 16: number l; LD 32: number l / 2.
 template <int LD>
-__device__ __forceinline__ float os_reduce8(float (&a)[8], int l) {
+__device__ __forceinline__ void os_reduce16(float (&a)[16], int l) {
     int o = LD / 2;
 #pragma unroll
-    for (int half = 4; half >= 1; half >>= 1, o >>= 1) {
+    for (int half = 8; half >= 1; half >>= 1, o >>= 1) {
+        if (o == 0) break;
         const bool up = (l & o) != 0;
 #pragma unroll
         for (int j = 0; j < half; ++j) {
@@ -72,11 +76,18 @@ __device__ __forceinline__ float os_reduce8(float (&a)[8], int l) {
             a[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
         }
     }
-    float s = a[0];
-#pragma unroll
-    for (; o >= 1; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    return s;
+    if (LD == 32) a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
 }
+
+// named barriers of the hand-over (0 is __syncthreads): all five warps take part
+__device__ __forceinline__ void os_bar_sync(int id) {
+    asm volatile("bar.sync %0, %1;" ::"r"(id), "n"(OS_THREADS + 32) : "memory");
+}
+__device__ __forceinline__ void os_bar_arrive(int id) {
+    asm volatile("bar.arrive %0, %1;" ::"r"(id), "n"(OS_THREADS + 32) : "memory");
+}
+#define OS_FULL(stage) (1 + (stage))
+#define OS_EMPTY(stage) (1 + OS_STAGES + (stage))
 
 // One token on this thread's two columns: acc += (state read with r), state updated.
 template <int ND4, bool WKV>
@@ -115,90 +126,164 @@ __device__ __forceinline__ void os_token(float4 (&S0)[ND4], float4 (&S1)[ND4], c
 __device__ __forceinline__ float os_soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 
 // LD: lanes that share a pair of columns; ND4: float4 groups of a column a lane holds (D <= 4 LD ND4);
-// tc: tokens of a chunk (mlstm: at most 32)
+// tc: tokens of a chunk
 template <int LD, int ND4, bool WKV>
-__global__ void __launch_bounds__(OS_THREADS) outer_scan_kernel(OuterScanArgs a, int tc) {
+__global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanArgs a, int tc) {
     pdl_launch_dependents();
     constexpr int DP = 4 * LD * ND4;                   // padded key size
     constexpr int TV = 2 * (OS_THREADS / LD);          // columns of a block
     constexpr int NVEC = WKV ? 3 : 2;                  // vectors staged per token: r, k (and decays)
     extern __shared__ __align__(16) float os_smem[];
-    const int buf_floats = tc * (NVEC * DP + TV) + (WKV ? 0 : 2 * tc);   // r k (w) | v | raw i, f
-    float* o_s = os_smem + 2 * buf_floats;             // [tc][TV]
-    float* keep_s = o_s + tc * TV;                     // [tc] mlstm: decay of the state; wkv: r . (u k)
-    float* add_s = keep_s + tc;                        // [tc] mlstm: factor on the new term
-    float* floor_s = add_s + tc;                       // [tc] mlstm: e^(-m)
+    // a stage: r k (w) | v | factors: wkv r . (u k), mlstm (decay, input) pairs and e^(-m)
+    const int stage_floats = tc * (NVEC * DP + TV) + 4 * ((3 * tc + 3) / 4);
     const int D = a.D, Dv = a.Dv;
     const int cols = WKV ? Dv : Dv + 1;
     const int tiles = (cols + TV - 1) / TV;
     const int h = blockIdx.x / tiles, tile = blockIdx.x - h * tiles;
     const int b = blockIdx.y;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int l = tid % LD, c = tid / LD;              // lane of the pair's group; pair of columns
     const int j0 = tile * TV, n_cols = min(TV, cols - j0);
-    const bool live0 = 2 * c < n_cols, live1 = 2 * c + 1 < n_cols;
     const int t0 = a.cu_seqlens[b], n_b = a.cu_seqlens[b + 1] - t0;
     const int slot = a.slots[b];
-    // (a row of a tensor may start anywhere: 16-byte copies only where all of them start on 16 bytes)
-    const bool vec = (D & 3) == 0 &&
-                     ((a.r_width | a.k_width | a.w_width | (long long)(a.r_off | a.k_off | a.w_off)) & 3) == 0 &&
-                     (((uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.w) & 15) == 0;
-    if (DP > D) {                                      // the copies never touch the padding
-        const int pad = DP - D;
-        for (int i = tid; i < 2 * tc * NVEC * pad; i += OS_THREADS) {
-            const int row = i / pad, d = D + i - row * pad;
-            const int buf = row / (tc * NVEC), rr = row - buf * tc * NVEC;
-            os_smem[buf * buf_floats + rr * DP + d] = 0.0f;
-        }
-    }
-    float ib = 0.f, fb = 0.f;
-    if (!WKV) { ib = a.i_bias[h]; fb = a.f_bias[h]; }
-    pdl_wait();
-    if (n_b <= 0) return;
+    const int n_chunks = (n_b + tc - 1) / tc;
+    if (n_b <= 0) { pdl_wait(); return; }
 
-    auto fetch = [&](int c0, int buf) {
-        const int nc = min(tc, n_b - c0);
-        float* r_s = os_smem + buf * buf_floats;
-        float* k_s = r_s + tc * DP;
-        float* w_s = k_s + tc * DP;                    // (wkv)
-        float* v_s = r_s + tc * NVEC * DP;
-        if (vec) {
-            const int qn = D >> 2;
-            for (int i = tid; i < nc * qn; i += OS_THREADS) {
-                const int tt = i / qn, d = (i - tt * qn) << 2;
-                const size_t t = (size_t)(t0 + c0 + tt);
-                os_cp16(r_s + tt * DP + d, a.r + t * a.r_width + a.r_off + h * D + d);
-                os_cp16(k_s + tt * DP + d, a.k + t * a.k_width + a.k_off + h * D + d);
-                if (WKV) os_cp16(w_s + tt * DP + d, a.w + t * a.w_width + a.w_off + h * D + d);
-            }
-        } else {
-            for (int i = tid; i < nc * D; i += OS_THREADS) {
-                const int tt = i / D, d = i - tt * D;
-                const size_t t = (size_t)(t0 + c0 + tt);
-                os_cp4(r_s + tt * DP + d, a.r + t * a.r_width + a.r_off + h * D + d);
-                os_cp4(k_s + tt * DP + d, a.k + t * a.k_width + a.k_off + h * D + d);
-                if (WKV) os_cp4(w_s + tt * DP + d, a.w + t * a.w_width + a.w_off + h * D + d);
+    if (warp == OS_THREADS / 32) {
+        // ---- the feeding warp ----------------------------------------------------------------------
+        // (a row of a tensor may start anywhere: 16-byte copies only where all of them start on 16 bytes)
+        const bool vec = (D & 3) == 0 &&
+                         ((a.r_width | a.k_width | a.w_width | (long long)(a.r_off | a.k_off | a.w_off)) & 3) == 0 &&
+                         (((uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.w) & 15) == 0;
+        const bool vec_v = (Dv & 3) == 0 && ((a.v_width | (long long)a.v_off) & 3) == 0 && ((uintptr_t)a.v & 15) == 0;
+        if (DP > D) {                                  // the copies never touch the padding
+            const int pad = DP - D;
+            for (int i = lane; i < OS_STAGES * tc * NVEC * pad; i += 32) {
+                const int row = i / pad, d = D + i - row * pad;
+                const int st = row / (tc * NVEC), rr = row - st * tc * NVEC;
+                os_smem[st * stage_floats + rr * DP + d] = 0.0f;
             }
         }
-        for (int i = tid; i < nc * n_cols; i += OS_THREADS) {
-            const int tt = i / n_cols, cc = i - tt * n_cols;
-            if (WKV || j0 + cc < Dv)
-                os_cp4(v_s + tt * TV + cc, a.v + (size_t)(t0 + c0 + tt) * a.v_width + a.v_off + (size_t)h * Dv + j0 + cc);
-            else
-                v_s[tt * TV + cc] = 1.0f;              // the normalizer's column
-        }
-        if (!WKV) {
-            float* g_s = v_s + tc * TV;
-            for (int i = tid; i < 2 * nc; i += OS_THREADS) {
-                const int tt = i >> 1;
-                os_cp4(g_s + (i & 1) * tc + tt,
-                       a.gates + (size_t)(t0 + c0 + tt) * a.gate_width + ((i & 1) ? a.f_off : a.i_off) + h);
+        float ib = 0.f, fb = 0.f;
+        if (!WKV) { ib = a.i_bias[h]; fb = a.f_bias[h]; }
+        pdl_wait();
+        float m_run = 0.f;
+        if (!WKV) m_run = a.maxima[((size_t)slot * a.heads + h) * cols + j0];
+        float next_i = 0.f, next_f = 0.f;              // raw gates of the chunk asked for last
+        const int v_cols = min(n_cols, Dv - j0);       // columns of the tile that have values (may be 0)
+        auto fetch = [&](int chunk) {
+            const int c0 = chunk * tc, nc = min(tc, n_b - c0);
+            float* r_s = os_smem + (chunk % OS_STAGES) * stage_floats;
+            float* k_s = r_s + tc * DP;
+            float* w_s = k_s + tc * DP;                // (wkv)
+            float* v_s = r_s + tc * NVEC * DP;
+            const size_t t = (size_t)(t0 + c0);
+            const float* rg = a.r + t * a.r_width + a.r_off + h * D;
+            const float* kg = a.k + t * a.k_width + a.k_off + h * D;
+            const float* wg = WKV ? a.w + t * a.w_width + a.w_off + h * D : nullptr;
+            const float* vg = a.v + t * a.v_width + a.v_off + (size_t)h * Dv + j0;
+            for (int tt = 0; tt < nc; ++tt) {
+                if (vec) {
+                    for (int d = 4 * lane; d < D; d += 128) {
+                        os_cp16(r_s + d, rg + d);
+                        os_cp16(k_s + d, kg + d);
+                        if (WKV) os_cp16(w_s + d, wg + d);
+                    }
+                } else {
+                    for (int d = lane; d < D; d += 32) {
+                        os_cp4(r_s + d, rg + d);
+                        os_cp4(k_s + d, kg + d);
+                        if (WKV) os_cp4(w_s + d, wg + d);
+                    }
+                }
+                r_s += DP; k_s += DP; w_s += DP;
+                rg += a.r_width; kg += a.k_width; if (WKV) wg += a.w_width;
             }
-        }
+            if (vec_v && (v_cols & 3) == 0) {
+                const int per = v_cols >> 2;
+                for (int i = lane; i < nc * per; i += 32) {
+                    const int tt = i / per, cc = (i - tt * per) << 2;
+                    os_cp16(v_s + tt * TV + cc, vg + (size_t)tt * a.v_width + cc);
+                }
+            } else {
+                for (int i = lane; i < nc * v_cols; i += 32) {
+                    const int tt = i / v_cols, cc = i - tt * v_cols;
+                    os_cp4(v_s + tt * TV + cc, vg + (size_t)tt * a.v_width + cc);
+                }
+            }
+            if (!WKV) {
+                if (j0 + n_cols == cols)               // the normalizer's column
+                    for (int tt = lane; tt < nc; tt += 32) v_s[tt * TV + n_cols - 1] = 1.0f;
+                if (lane < nc) {
+                    const float* g = a.gates + (t + lane) * a.gate_width + h;
+                    next_i = g[a.i_off];
+                    next_f = g[a.f_off];
+                }
+            }
+        };
+        fetch(0);
         asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    fetch(0, 0);
+        for (int chunk = 0; chunk < n_chunks; ++chunk) {
+            const int nc = min(tc, n_b - chunk * tc);
+            const float raw_i = next_i, raw_f = next_f;
+            if (chunk + 1 < n_chunks) {
+                if (chunk + 1 >= OS_STAGES) os_bar_sync(OS_EMPTY((chunk + 1) % OS_STAGES));
+                fetch(chunk + 1);
+            }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+            __syncwarp();                              // every lane's copies of this chunk are there
+            float* r_s = os_smem + (chunk % OS_STAGES) * stage_floats;
+            float* k_s = r_s + tc * DP;
+            float* f_s = r_s + tc * (NVEC * DP + TV);
+            if (WKV) {
+                // r . (u k): what the current token's own value is multiplied by
+                float s[16];
+#pragma unroll
+                for (int tt = 0; tt < 16; ++tt) s[tt] = 0.f;
+                for (int d = lane; d < D; d += 32) {
+                    const float ud = a.u[h * D + d];
+#pragma unroll
+                    for (int tt = 0; tt < 16; ++tt)
+                        if (tt < nc) s[tt] = fmaf(r_s[tt * DP + d] * ud, k_s[tt * DP + d], s[tt]);
+                }
+                os_reduce16<32>(s, lane);
+                if ((lane & 1) == 0 && (lane >> 1) < nc) f_s[lane >> 1] = s[0];
+            } else {
+                // a token a lane; the maxima by a scan in which a stretch of tokens is the pair
+                // (sum of f, largest i + the f's after it)
+                const bool mine = lane < nc;
+                const float li = mine ? os_soft_cap(raw_i + ib, a.cap) : -INFINITY;
+                const float zf = mine ? os_soft_cap(raw_f + fb, a.cap) : 0.f;
+                const float lf = mine ? fminf(zf, 0.f) - log1pf(expf(-fabsf(zf))) : 0.f;
+                float F = lf, M = li;
+#pragma unroll
+                for (int o = 1; o < OS_TC; o <<= 1) {
+                    const float pF = __shfl_up_sync(0xffffffffu, F, o), pM = __shfl_up_sync(0xffffffffu, M, o);
+                    if (lane >= o) { M = fmaxf(pM + F, M); F = pF + F; }
+                }
+                const float m_t = fmaxf(F + m_run, M);
+                float before = __shfl_up_sync(0xffffffffu, m_t, 1);
+                if (lane == 0) before = m_run;
+                if (mine) {
+                    // (m_t is often lf + before, rounded: in this order the difference is exact, so what m_t
+                    // lost in rounding stays in the state's factor instead of adding up token by token)
+                    f_s[2 * lane] = expf((before - m_t) + lf);
+                    f_s[2 * lane + 1] = expf(li - m_t);
+                    f_s[2 * tc + lane] = expf(-m_t);
+                }
+                m_run = __shfl_sync(0xffffffffu, m_t, nc - 1);
+            }
+            os_bar_arrive(OS_FULL(chunk % OS_STAGES));
+        }
+        if (!WKV)
+            for (int i = lane; i < n_cols; i += 32) a.maxima[((size_t)slot * a.heads + h) * cols + j0 + i] = m_run;
+        return;
+    }
 
+    // ---- the four warps that walk the tokens ---------------------------------------------------------
+    const int l = tid % LD, c = tid / LD;              // lane of the pair's group; pair of columns
+    const bool live0 = 2 * c < n_cols, live1 = 2 * c + 1 < n_cols;
+    pdl_wait();
     float* st0 = a.state + (((size_t)slot * a.heads + h) * cols + j0 + (live0 ? 2 * c : 0)) * D;
     float* st1 = live1 ? st0 + D : st0;
     float4 S0[ND4], S1[ND4];
@@ -222,108 +307,72 @@ __global__ void __launch_bounds__(OS_THREADS) outer_scan_kernel(OuterScanArgs a,
         S0[i] = get(st0, 4 * (l + LD * i), live0);
         S1[i] = get(st1, 4 * (l + LD * i), live1);
     }
-    float m_run = 0.f;                                 // (warp 0) the running maximum
-    if (!WKV) m_run = a.maxima[((size_t)slot * a.heads + h) * cols + j0];
-
-    for (int c0 = 0, buf = 0; c0 < n_b; c0 += tc, buf ^= 1) {
-        const int nc = min(tc, n_b - c0);
-        if (c0 + tc < n_b) {
-            fetch(c0 + tc, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();                 // the chunk has arrived; the last chunk's outputs are written
-        const float* r_s = os_smem + buf * buf_floats;
-        const float* k_s = r_s + tc * DP;
-        const float* w_s = k_s + tc * DP;
+    const size_t out_row = (size_t)a.heads * Dv;
+    float* out0 = a.out + (size_t)t0 * out_row + (size_t)h * Dv + j0;
+    // number `x` is the sum of token t (of the chunk, whose first token's output row is o) and column cc
+    auto emit = [&](float x, float* o, const float* v_s, const float* f_s, int t, int cc, int token) {
+        if (cc >= n_cols) return;
+        if (WKV) o[t * out_row + cc] = fmaf(f_s[t], v_s[t * TV + cc], x);
+        else if (j0 + cc < Dv) o[t * out_row + cc] = x * a.r_scale;
+        else a.den[(size_t)(token + t) * a.heads + h] = fmaxf(fabsf(x * a.r_scale), f_s[2 * tc + t]) + 1e-6f;
+    };
+    for (int chunk = 0; chunk < n_chunks; ++chunk) {
+        const int stage = chunk % OS_STAGES;
+        const int nc = min(tc, n_b - chunk * tc);
+        os_bar_sync(OS_FULL(stage));
+        const float* r_s = os_smem + stage * stage_floats;
         const float* v_s = r_s + tc * NVEC * DP;
-        if (WKV) {
-            // r . (u k): what the current token's own value is multiplied by
-            for (int tt = warp; tt < nc; tt += OS_THREADS / 32) {
-                float s = 0.f;
-                for (int d = lane; d < D; d += 32)
-                    s = fmaf(r_s[tt * DP + d] * a.u[h * D + d], k_s[tt * DP + d], s);
-                s = warp_sum(s);
-                if (lane == 0) keep_s[tt] = s;
-            }
-        } else if (warp == 0) {
-            // the gates of the chunk's tokens, a lane each; the maxima by a scan in which a stretch
-            // of tokens is the pair (sum of f, largest i + the f's after it)
-            const float* g_s = v_s + tc * TV;
-            const bool mine = lane < nc;
-            const float li = mine ? os_soft_cap(g_s[lane] + ib, a.cap) : -INFINITY;
-            const float zf = mine ? os_soft_cap(g_s[tc + lane] + fb, a.cap) : 0.f;
-            const float lf = mine ? fminf(zf, 0.f) - log1pf(expf(-fabsf(zf))) : 0.f;
-            float F = lf, M = li;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float pF = __shfl_up_sync(0xffffffffu, F, o), pM = __shfl_up_sync(0xffffffffu, M, o);
-                if (lane >= o) { M = fmaxf(pM + F, M); F = pF + F; }
-            }
-            const float m_t = fmaxf(F + m_run, M);
-            float before = __shfl_up_sync(0xffffffffu, m_t, 1);
-            if (lane == 0) before = m_run;
-            if (mine) {
-                // (m_t is often lf + before, rounded: in this order the difference is exact, so what m_t lost
-                // in rounding stays in the state's factor instead of adding up token by token)
-                keep_s[lane] = expf((before - m_t) + lf);
-                add_s[lane] = expf(li - m_t);
-                floor_s[lane] = expf(-m_t);
-            }
-            m_run = __shfl_sync(0xffffffffu, m_t, nc - 1);
-        }
-        if (!WKV) __syncthreads();       // (wkv reads its factors after the tokens, behind a barrier)
+        const float* f_s = v_s + tc * TV;
+        const float4* r4 = reinterpret_cast<const float4*>(r_s) + l;
+        const float4* k4 = r4 + tc * (DP / 4);
+        const float4* w4 = k4 + tc * (DP / 4);
+        float* o = out0 + (size_t)chunk * tc * out_row;
+        const int token = t0 + chunk * tc;
         int tt = 0;
         for (; tt + OS_TU <= nc; tt += OS_TU) {
             float acc[2 * OS_TU];
 #pragma unroll
             for (int u = 0; u < OS_TU; ++u) {
                 const int t = tt + u;
-                const float2 vv = *reinterpret_cast<const float2*>(v_s + t * TV + 2 * c);
-                float v0 = live0 ? vv.x : 0.f, v1 = live1 ? vv.y : 0.f, keep = 0.f;
-                if (!WKV) { keep = keep_s[t]; v0 *= add_s[t]; v1 *= add_s[t]; }
-                os_token<ND4, WKV>(S0, S1, reinterpret_cast<const float4*>(r_s + t * DP) + l,
-                                   reinterpret_cast<const float4*>(k_s + t * DP) + l,
-                                   reinterpret_cast<const float4*>(w_s + t * DP) + l, keep, v0, v1, LD,
+                float2 vv = *reinterpret_cast<const float2*>(v_s + t * TV + 2 * c);
+                float keep = 0.f;
+                if (!WKV) {
+                    const float2 f = *reinterpret_cast<const float2*>(f_s + 2 * t);
+                    keep = f.x; vv.x *= f.y; vv.y *= f.y;
+                }
+                os_token<ND4, WKV>(S0, S1, r4 + t * (DP / 4), k4 + t * (DP / 4), w4 + t * (DP / 4), keep, vv.x, vv.y, LD,
                                    acc[2 * u], acc[2 * u + 1]);
             }
-            const float sum = os_reduce8<LD>(acc, l);
-            constexpr int PER = LD / 8;                // lanes that hold the same sum
-            if (l % PER == 0) {
-                const int i = l / PER;
-                o_s[(tt + (i >> 1)) * TV + 2 * c + (i & 1)] = sum;
+            os_reduce16<LD>(acc, l);
+            if (LD == 8) {
+                emit(acc[0], o, v_s, f_s, tt + l, 2 * c, token);
+                emit(acc[1], o, v_s, f_s, tt + l, 2 * c + 1, token);
+            } else if (LD == 16) {
+                emit(acc[0], o, v_s, f_s, tt + (l >> 1), 2 * c + (l & 1), token);
+            } else if ((l & 1) == 0) {
+                emit(acc[0], o, v_s, f_s, tt + (l >> 2), 2 * c + ((l >> 1) & 1), token);
             }
         }
         for (; tt < nc; ++tt) {
-            const float2 vv = *reinterpret_cast<const float2*>(v_s + tt * TV + 2 * c);
-            float v0 = live0 ? vv.x : 0.f, v1 = live1 ? vv.y : 0.f, keep = 0.f, a0, a1;
-            if (!WKV) { keep = keep_s[tt]; v0 *= add_s[tt]; v1 *= add_s[tt]; }
-            os_token<ND4, WKV>(S0, S1, reinterpret_cast<const float4*>(r_s + tt * DP) + l,
-                               reinterpret_cast<const float4*>(k_s + tt * DP) + l,
-                               reinterpret_cast<const float4*>(w_s + tt * DP) + l, keep, v0, v1, LD, a0, a1);
-#pragma unroll
-            for (int o = LD / 2; o > 0; o >>= 1) {
-                a0 += __shfl_xor_sync(0xffffffffu, a0, o);
-                a1 += __shfl_xor_sync(0xffffffffu, a1, o);
+            float2 vv = *reinterpret_cast<const float2*>(v_s + tt * TV + 2 * c);
+            float keep = 0.f, a0, a1;
+            if (!WKV) {
+                const float2 f = *reinterpret_cast<const float2*>(f_s + 2 * tt);
+                keep = f.x; vv.x *= f.y; vv.y *= f.y;
             }
-            if (l == 0) { o_s[tt * TV + 2 * c] = a0; o_s[tt * TV + 2 * c + 1] = a1; }
+            os_token<ND4, WKV>(S0, S1, r4 + tt * (DP / 4), k4 + tt * (DP / 4), w4 + tt * (DP / 4), keep, vv.x, vv.y, LD, a0, a1);
+#pragma unroll
+            for (int o2 = LD / 2; o2 > 0; o2 >>= 1) {
+                a0 += __shfl_xor_sync(0xffffffffu, a0, o2);
+                a1 += __shfl_xor_sync(0xffffffffu, a1, o2);
+            }
+            if (l == 0) {
+                emit(a0, o, v_s, f_s, tt, 2 * c, token);
+                emit(a1, o, v_s, f_s, tt, 2 * c + 1, token);
+            }
         }
-        __syncthreads();                 // the chunk's outputs are complete; its buffer may be refilled
-        for (int i = tid; i < nc * n_cols; i += OS_THREADS) {
-            const int t2 = i / n_cols, cc = i - t2 * n_cols;
-            const size_t t = (size_t)(t0 + c0 + t2);
-            const float x = o_s[t2 * TV + cc];
-            if (WKV)
-                a.out[t * a.heads * Dv + (size_t)h * Dv + j0 + cc] = fmaf(keep_s[t2], v_s[t2 * TV + cc], x);
-            else if (j0 + cc < Dv)
-                a.out[t * a.heads * Dv + (size_t)h * Dv + j0 + cc] = x * a.r_scale;
-            else
-                a.den[t * a.heads + h] = fmaxf(fabsf(x * a.r_scale), floor_s[t2]) + 1e-6f;
-        }
-        // (the next chunk's copies go to the other buffer, and its factors are formed behind the
-        // barrier at the head of the loop)
-        if (WKV && c0 + tc < n_b) __syncthreads();     // its v is about to be the target of the copy after next
+        // (only a stage that will be filled again is handed back: nobody waits for the others)
+        if (chunk + OS_STAGES < n_chunks) os_bar_arrive(OS_EMPTY(stage));
     }
     auto put = [&](float* p, int d, const float4& x) {
         if (vec_state) {
@@ -340,48 +389,48 @@ __global__ void __launch_bounds__(OS_THREADS) outer_scan_kernel(OuterScanArgs a,
         if (live0) put(st0, 4 * (l + LD * i), S0[i]);
         if (live1) put(st1, 4 * (l + LD * i), S1[i]);
     }
-    if (!WKV && warp == 0)
-        for (int i = lane; i < n_cols; i += 32) a.maxima[((size_t)slot * a.heads + h) * cols + j0 + i] = m_run;
 }
 
 template <int LD, int ND4, bool WKV>
-static int os_launch(const OuterScanArgs& a, cudaStream_t stream) {
+static int os_launch(const OuterScanArgs& a, int max_tokens, cudaStream_t stream) {
     constexpr int DP = 4 * LD * ND4, TV = 2 * (OS_THREADS / LD), NVEC = WKV ? 3 : 2;
-    const int tc = DP > 128 ? 16 : 32;
-    const size_t smem = (size_t)(2 * (tc * (NVEC * DP + TV) + (WKV ? 0 : 2 * tc)) + tc * TV + 3 * tc) * sizeof(float);
+    // (short rows take shorter chunks, so that more blocks fit an SM: single tokens most of all)
+    const int tc = max_tokens < 1 ? OS_TC : max_tokens < OS_TC ? max_tokens : OS_TC;
+    auto bytes = [&](int t) { return (size_t)OS_STAGES * (t * (NVEC * DP + TV) + 4 * ((3 * t + 3) / 4)) * sizeof(float); };
     static bool configured[64] = {false};
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return MF_ERR_UNSUPPORTED;
     if (!configured[dev]) {
         cudaError_t e = cudaFuncSetAttribute(outer_scan_kernel<LD, ND4, WKV>,
-                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes(OS_TC));
         if (e != cudaSuccess) return (int)e;
         configured[dev] = true;
     }
     const int cols = WKV ? a.Dv : a.Dv + 1;
     const int tiles = (cols + TV - 1) / TV;
-    mf_launch(outer_scan_kernel<LD, ND4, WKV>, dim3(a.heads * tiles, a.n_rows), dim3(OS_THREADS), smem,
+    mf_launch(outer_scan_kernel<LD, ND4, WKV>, dim3(a.heads * tiles, a.n_rows), dim3(OS_THREADS + 32), bytes(tc),
               stream, a, tc);
     return MF_LAUNCH_CHECK();
 }
 
 template <bool WKV>
-static int os_choose(const OuterScanArgs& a, cudaStream_t stream) {
+static int os_choose(const OuterScanArgs& a, int max_tokens, cudaStream_t stream) {
     if (a.n_rows <= 0) return 0;
     if (a.D < 1 || a.D > OS_MAX_D || a.Dv < 1 || a.heads < 1 || a.n_rows > 65535) return MF_ERR_UNSUPPORTED;
     if (((uintptr_t)a.state & 15) != 0) return MF_ERR_UNSUPPORTED;
-    if (a.D <= 32) return os_launch<8, 1, WKV>(a, stream);
-    if (a.D <= 64) return os_launch<16, 1, WKV>(a, stream);
-    if (a.D <= 128) return os_launch<16, 2, WKV>(a, stream);
-    return os_launch<32, 2, WKV>(a, stream);
+    if (a.D <= 32) return os_launch<8, 1, WKV>(a, max_tokens, stream);
+    if (a.D <= 64) return os_launch<16, 1, WKV>(a, max_tokens, stream);
+    if (a.D <= 128) return os_launch<16, 2, WKV>(a, max_tokens, stream);
+    return os_launch<32, 2, WKV>(a, max_tokens, stream);
 }
 
-extern "C" int mf_wkv_scan(const OuterScanArgs* args, cudaStream_t stream) {
-    return os_choose<true>(*args, stream);
+// max_tokens: the most tokens a row brings (0: not known; it only sizes the chunks)
+extern "C" int mf_wkv_scan(const OuterScanArgs* args, int max_tokens, cudaStream_t stream) {
+    return os_choose<true>(*args, max_tokens, stream);
 }
-extern "C" int mf_mlstm_scan(const OuterScanArgs* args, cudaStream_t stream) {
+extern "C" int mf_mlstm_scan(const OuterScanArgs* args, int max_tokens, cudaStream_t stream) {
     if (!(args->cap > 0.0f)) return MF_ERR_ARGUMENT;
-    return os_choose<false>(*args, stream);
+    return os_choose<false>(*args, max_tokens, stream);
 }
 
 // ------------------------------------------------------------------------------------------
@@ -395,11 +444,12 @@ __global__ void __launch_bounds__(128)
 wkv_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* __restrict__ w2t,
                  const float* __restrict__ w0, float* __restrict__ out, int n_tokens, int rank, int channels) {
     pdl_prologue();
-    extern __shared__ float wd_s[];                    // [NT][rank]
+    extern __shared__ __align__(16) float wd_s[];      // [NT][rank, padded to a multiple of 4]
     const int first = blockIdx.y * NT, nt = min(NT, n_tokens - first);
+    const int pitch = (rank + 3) & ~3;
     for (int i = threadIdx.x; i < NT * rank; i += blockDim.x) {
         const int t = i / rank, r = i - t * rank;
-        wd_s[i] = t < nt ? tanhf(t1[(size_t)(first + t) * t1_width + r]) : 0.f;
+        wd_s[t * pitch + r] = t < nt ? tanhf(t1[(size_t)(first + t) * t1_width + r]) : 0.f;
     }
     __syncthreads();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -408,11 +458,30 @@ wkv_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* 
     const float base = w0[c];
 #pragma unroll
     for (int t = 0; t < NT; ++t) acc[t] = base;
-#pragma unroll 4
-    for (int r = 0; r < rank; ++r) {
+    int r = 0;
+    // four numbers of the rank at a time (every row of wd_s starts on 16 bytes); few tokens: more of the
+    // matrix's loads in flight, since nothing else hides them
+    constexpr int AHEAD = NT <= 2 ? 4 : 1;
+    for (; r + 4 * AHEAD <= rank; r += 4 * AHEAD) {
+        float w[4 * AHEAD];
+#pragma unroll
+        for (int i = 0; i < 4 * AHEAD; ++i) w[i] = w2t[(size_t)(r + i) * channels + c];
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+#pragma unroll
+            for (int i = 0; i < AHEAD; ++i) {
+                const float4 x = *reinterpret_cast<const float4*>(wd_s + t * pitch + r + 4 * i);
+                acc[t] = fmaf(w[4 * i], x.x, acc[t]);
+                acc[t] = fmaf(w[4 * i + 1], x.y, acc[t]);
+                acc[t] = fmaf(w[4 * i + 2], x.z, acc[t]);
+                acc[t] = fmaf(w[4 * i + 3], x.w, acc[t]);
+            }
+        }
+    }
+    for (; r < rank; ++r) {
         const float w = w2t[(size_t)r * channels + c];
 #pragma unroll
-        for (int t = 0; t < NT; ++t) acc[t] = fmaf(w, wd_s[t * rank + r], acc[t]);
+        for (int t = 0; t < NT; ++t) acc[t] = fmaf(w, wd_s[t * pitch + r], acc[t]);
     }
 #pragma unroll
     for (int t = 0; t < NT; ++t)
@@ -422,16 +491,16 @@ wkv_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* 
 extern "C" int mf_wkv_decay(const float* t1, long long t1_width, const float* w2t, const float* w0,
                             float* out, int n_tokens, int rank, int channels, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (rank < 1 || channels < 1 || (size_t)rank * WD_T * sizeof(float) > 48 * 1024) return MF_ERR_UNSUPPORTED;
+    if (rank < 1 || channels < 1 || (size_t)(rank + 3) * WD_T * sizeof(float) > 48 * 1024) return MF_ERR_UNSUPPORTED;
     const int cb = (channels + 127) / 128;
     if (n_tokens <= 64) {
         if ((n_tokens + 1) / 2 > 65535) return MF_ERR_UNSUPPORTED;
-        mf_launch(wkv_decay_kernel<2>, dim3(cb, (n_tokens + 1) / 2), dim3(128), (size_t)rank * 2 * sizeof(float),
+        mf_launch(wkv_decay_kernel<2>, dim3(cb, (n_tokens + 1) / 2), dim3(128), (size_t)((rank + 3) & ~3) * 2 * sizeof(float),
                   stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels);
     } else {
         if ((n_tokens + WD_T - 1) / WD_T > 65535) return MF_ERR_UNSUPPORTED;
         mf_launch(wkv_decay_kernel<WD_T>, dim3(cb, (n_tokens + WD_T - 1) / WD_T), dim3(128),
-                  (size_t)rank * WD_T * sizeof(float), stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels);
+                  (size_t)((rank + 3) & ~3) * WD_T * sizeof(float), stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels);
     }
     return MF_LAUNCH_CHECK();
 }

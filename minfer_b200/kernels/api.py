@@ -243,8 +243,8 @@ def _sig_retention(lib: ctypes.CDLL) -> None:
 
 
 def _sig_outer_scan(lib: ctypes.CDLL) -> None:
-    lib.mf_wkv_scan.argtypes = [c_void_p, c_void_p]
-    lib.mf_mlstm_scan.argtypes = [c_void_p, c_void_p]
+    lib.mf_wkv_scan.argtypes = [c_void_p, c_int, c_void_p]
+    lib.mf_mlstm_scan.argtypes = [c_void_p, c_int, c_void_p]
     lib.mf_wkv_decay.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                  c_int, c_void_p]
 
@@ -289,6 +289,8 @@ def _sig_moe(lib: ctypes.CDLL) -> None:
     lib.mf_moe_place.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                  c_void_p]
     lib.mf_moe_gather.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
+    lib.mf_moe_group_few.argtypes = [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
+                                     c_void_p, c_void_p]
     lib.mf_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                    c_int, c_void_p]
 
@@ -1382,6 +1384,20 @@ def moe_place(idx: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor, or
                                     _stream()), "moe_place", 2)
 
 
+def moe_group_few(idx: torch.Tensor, x: torch.Tensor, experts: int, out: torch.Tensor, offsets: torch.Tensor,
+                  where: torch.Tensor) -> None:
+    """``moe_counts``, ``moe_place`` and ``moe_gather`` in one launch for up to 4,096 (token, choice) pairs:
+    the pairs of ``idx`` [tokens, top] grouped by expert, offsets[e] = first row of expert e, where[pair] =
+    the pair's row, out[where[pair]] = x[pair's token] (rows of a multiple of 16 bytes)."""
+    n, top = idx.shape
+    if (out.shape != (n * top, x.shape[1]) or out.dtype != x.dtype or offsets.numel() != experts + 1
+            or where.numel() != n * top or x.shape[0] != n):
+        raise KernelError("moe_group_few: shapes do not fit")
+    _check(_lib("moe").mf_moe_group_few(
+        _i32(idx, "idx"), n * top, int(experts), top, _ptr(x, "x"), _ptr(out, "out"),
+        x.shape[1] * x.element_size(), _i32(offsets, "offsets"), _i32(where, "where"), _stream()), "moe_group_few")
+
+
 def moe_gather(x: torch.Tensor, pairs: torch.Tensor, out: torch.Tensor, top: int) -> None:
     """out[i] = x[pairs[i] // top]: the rows of the tokens behind the (token, choice) pairs."""
     if out.shape != (pairs.numel(), x.shape[1]) or out.dtype != x.dtype:
@@ -1675,10 +1691,11 @@ def wkv_decay(t1: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, out: torch.
 
 def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor,
              state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
-             n_rows: int) -> None:
+             n_rows: int, max_tokens: int = 0) -> None:
     """Per (row, head), tokens one after another: out = S^T r + (r . (bonus k)) v, then
     S <- diag(decay) S + k v^T.  ``r``, ``k``, ``decay`` float32 [tokens, heads * D], ``v`` and ``out``
-    [tokens, heads * Dv], ``bonus`` [heads, D]; S float32 in ``state`` [slots, heads, Dv, D]."""
+    [tokens, heads * Dv], ``bonus`` [heads, D]; S float32 in ``state`` [slots, heads, Dv, D].
+    ``max_tokens``: the most tokens a row brings (0: not known)."""
     n = r.shape[0]
     _, heads, dv, d = state.shape
     if (r.shape != (n, heads * d) or k.shape != r.shape or decay.shape != r.shape
@@ -1692,13 +1709,13 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Ten
     a.v_width = heads * dv
     a.n_rows, a.heads, a.D, a.Dv = int(n_rows), heads, d, dv
     a.r_scale = 1.0
-    _check(_lib("outer_scan").mf_wkv_scan(ctypes.addressof(a), _stream()), "wkv_scan")
+    _check(_lib("outer_scan").mf_wkv_scan(ctypes.addressof(a), int(max_tokens), _stream()), "wkv_scan")
 
 
 def mlstm_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off: int, f_off: int,
                i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, q_scale: float,
                state: torch.Tensor, maxima: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
-               out: torch.Tensor, den: torch.Tensor, n_rows: int) -> None:
+               out: torch.Tensor, den: torch.Tensor, n_rows: int, max_tokens: int = 0) -> None:
     """The matrix memory with exponential gates per (row, head), tokens one after another, from the
     columns of the float32 rows ``proj``: q and k (heads of D), v (heads of Dv), the raw input and
     forget gates (one per head).  ``out`` [tokens, heads * Dv] = S^T q (q times ``q_scale``) and
@@ -1722,7 +1739,7 @@ def mlstm_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off: in
     a.out, a.den = _f32(out, "out"), _f32(den, "den")
     a.n_rows, a.heads, a.D, a.Dv = int(n_rows), heads, d, dv
     a.cap, a.r_scale = float(cap), float(q_scale)
-    _check(_lib("outer_scan").mf_mlstm_scan(ctypes.addressof(a), _stream()), "mlstm_scan")
+    _check(_lib("outer_scan").mf_mlstm_scan(ctypes.addressof(a), int(max_tokens), _stream()), "mlstm_scan")
 
 
 class _SelectiveArgs(ctypes.Structure):

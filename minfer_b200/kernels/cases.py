@@ -581,6 +581,48 @@ def zanelorn_step_decode(reps, batch=8, ctx=2048):
     print(f"zanelorn decode step, batch {batch} at {ctx} positions, six layers: {us:.1f} us")
 
 
+def _pikavik_engine(max_tokens=8 * 4096, max_seqs=8):
+    from ..engine.step import Engine
+    from ..model import Model
+    moe = {"kind": "moe", "expert": {"ff": 1408, "limit": 7.0}, "shared": {"ff": 1408, "limit": 7.0},
+           "router": {"experts": 32, "top": 4, "scale": 2.5, "groups": {"count": 8, "keep": 5}}}
+    mixers = [{"type": "wkv", "mixer": {"heads": 32, "dim": 64, "decay_rank": 64}},
+              {"type": "mlstm", "mixer": {"heads": 8, "dim": 128, "vdim": 256, "gate_cap": 15.0}},
+              {"type": "latent_attention",
+               "mixer": {"heads": 16, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 768,
+                         "scale": 128 ** -0.5, "rot": {"base": 100000.0, "dims": 64}}}]
+    cfg = {"architecture": "Pikavik", "vocab": 32000, "width": 2048, "norm": {"eps": 1e-6},
+           "layers": [dict(m, mlp=moe) for m in mixers]}
+    model = Model.from_config(cfg, seed=0, dtype="bfloat16", device="cuda:0", make_on="device")
+    return Engine(model, max_tokens=max_tokens, max_seqs=max_seqs, cuda_graphs=False), cfg
+
+
+def pikavik_step_prefill(reps, tokens=2048):
+    """A whole prompt of 2,048 tokens through a Pikavik model of width 2,048: three layers, WKV, mLSTM
+    and latent attention, each with routed experts, plus the head."""
+    eng, cfg = _pikavik_engine()
+    g = torch.Generator().manual_seed(0)
+    ids = torch.randint(0, cfg["vocab"], (tokens,), generator=g).tolist()
+
+    def run():
+        s = eng.acquire()
+        eng.step([s], [ids])
+        eng.release(s)
+    us = _time(run, reps, graph=False)
+    print(f"pikavik prefill step, {tokens} tokens, three layers: {us:.1f} us")
+
+
+def pikavik_step_decode(reps, batch=8, ctx=2048):
+    """Decode steps of 8 sequences at 2,048 positions through the same model, kernel by kernel."""
+    eng, cfg = _pikavik_engine()
+    g = torch.Generator().manual_seed(0)
+    slots = [eng.acquire() for _ in range(batch)]
+    eng.step(slots, [torch.randint(0, cfg["vocab"], (ctx,), generator=g).tolist() for _ in range(batch)])
+    tokens = torch.randint(0, cfg["vocab"], (batch,), dtype=torch.int32, device="cuda")
+    us = _time(lambda: eng.decode_on_device(slots, tokens), reps, graph=False)
+    print(f"pikavik decode step, batch {batch} at {ctx} positions, three layers: {us:.1f} us")
+
+
 CASES = {f.__name__: f for f in (gemm_decode, gemm_decode_split, gemm_decode_m64, gemm_decode_split_m64, gemm_prefill, gemm_prefill_down,
                                  gemm_decode_cluster, gemm_decode_cluster_o, gemm_decode_cluster_m64,
                                  attention_decode, attention_decode_b8, attention_decode_long, attention_prefill,
@@ -589,7 +631,8 @@ CASES = {f.__name__: f for f in (gemm_decode, gemm_decode_split, gemm_decode_m64
                                  step_prefill, step_prefill_timeline, step_portions, step_decode, step_decode_sweep, step_prefill_sweep, step_decode_timeline,
                                  step_decode_timeline_b64, step_decode_b64, step_decode_small,
                                  ssm_scan_prompt, ssm_scan_decode, budanex_step_prefill, budanex_step_decode,
-                                 zanelorn_step_prefill, zanelorn_step_decode)}
+                                 zanelorn_step_prefill, zanelorn_step_decode,
+                                 pikavik_step_prefill, pikavik_step_decode)}
 
 
 def main(argv=None) -> int:

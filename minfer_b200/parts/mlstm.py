@@ -108,7 +108,7 @@ class MLstm(Mixer):
         i_off = 2 * nq + 2 * nv
         K.mlstm_scan(proj, 0, nq, 2 * nq, i_off, i_off + nh, self.w["i.b"], self.w["f.b"], self.gate_cap,
                      self.head_dim ** -0.5, binding.state[MLSTM_STATE], binding.state[MLSTM_MAXIMUM],
-                     ctx.cu_seqlens, ctx.slots, o, den, ctx.n_rows)
+                     ctx.cu_seqlens, ctx.slots, o, den, ctx.n_rows, ctx.max_row_tokens)
         gated = torch.empty((n, nv), dtype=ctx.act_dtype, device=dev)
         K.unit_norm_gate(o, proj, 2 * nq + nv, gated, nh, self.norm_eps, "sigmoid", den=den,
                          weight=self.w["norm"])

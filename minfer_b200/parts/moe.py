@@ -28,9 +28,9 @@ Every size is a parameter, and so are the tensors' names (behind the layer's pre
 expert's number, followed by ``.gate``, ``.up``, ``.down``.  The experts' matrices are stacked at
 load ([experts, ff, width] and [experts, width, ff]).
 
-Two ways through a step.  Few tokens (decoding; always inside a CUDA graph capture): one kernel
-per half, a block per (token, choice), the expert's rows read by index; nothing is read back.  Many
-tokens: the (token, choice) pairs are grouped by expert on the device, and every expert runs as two
+Two ways through a step.  Few tokens (always inside a CUDA graph capture, unless the other way
+reads nothing back either): one kernel per half, a block per (token, choice), the expert's rows read by
+index; nothing is read back.  Many tokens: the (token, choice) pairs are grouped by expert on the device, and every expert runs as two
 dense products over its rows, the gate's activation in the first one's epilogue; the weighted rows are
 then added into the residual token by token, the choices in order, so the sum does not depend on the
 batch.  On the tensor cores the two products of all experts are two launches, whose blocks read the
@@ -52,6 +52,10 @@ from .sink_attention import project_out
 
 # steps of up to this many tokens run the per-token kernels
 PER_TOKEN_MAX = int(os.environ.get("MINFER_B200_MOE_PER_TOKEN_MAX", "48"))
+# ... unless the grouped products of the tensor cores take the sizes: then up to this many
+PER_TOKEN_MAX_GROUPED = int(os.environ.get("MINFER_B200_MOE_PER_TOKEN_MAX_GROUPED", "0"))
+# (token, choice) pairs that one launch groups and gathers
+GROUP_FEW_MAX = 1024
 
 
 class RoutedExperts(FeedForward):
@@ -115,8 +119,8 @@ class RoutedExperts(FeedForward):
         self.expert_name = expert_name
         self.init_std, self.router_std = float(init_std), float(router_std)
         # the per-token kernels keep a token's input and its experts' hidden values in shared memory;
-        # sizes beyond that always take the grouped path, which reads a few numbers back on the host
-        # and so cannot be part of a CUDA graph
+        # sizes beyond that always take the grouped path, which (but for grouped products on the tensor
+        # cores) reads a few numbers back on the host and so cannot be part of a CUDA graph
         self.per_token_fits = (4 * self.hidden_size <= 48 * 1024
                                and 4 * self.top * self.intermediate_size <= 48 * 1024)
         self.capturable = self.per_token_fits
@@ -195,6 +199,7 @@ class RoutedExperts(FeedForward):
         pairs = self.w_gate_up.view(self.n_experts, self.intermediate_size, 2, self.hidden_size)
         self.w_gate, self.w_up = pairs[:, :, 0], pairs[:, :, 1]
         self.w_down = torch.stack([weights[f"{p}.down"].to(dtype) for p in names]).contiguous()
+        self.capturable = self.per_token_fits or self._grouped_weights()
 
     def export(self, prefix: str) -> Dict[str, torch.Tensor]:
         out = {f"{prefix}{self.router_name}": self.router.weight[:self.n_outputs]}
@@ -242,12 +247,14 @@ class RoutedExperts(FeedForward):
                                self.weight_scale)
         else:
             K.moe_route(logits, idx, wts, self.top)
-        if self.per_token_fits and (n <= PER_TOKEN_MAX or torch.cuda.is_current_stream_capturing()):
+        grouped = x.dtype == torch.bfloat16 and self._grouped_weights()
+        if self.per_token_fits and (n <= (PER_TOKEN_MAX_GROUPED if grouped else PER_TOKEN_MAX)
+                                    or (not grouped and torch.cuda.is_current_stream_capturing())):
             hidden = torch.empty((n, self.top, self.intermediate_size), dtype=x.dtype, device=dev)
             K.moe_experts(x, self.w_gate, self.w_up, self.w_down, idx, wts, hidden, residual,
                           self.activation, self.limit, self.alpha, store=fresh)
         else:
-            self._grouped(x, idx, wts, residual, fresh)
+            self._grouped(x, idx, wts, residual, fresh, grouped)
         if self.shared is not None:
             # act(gate, up) * sigmoid(the router product's extra column), then down into the stream
             from ..kernels import gemm
@@ -270,32 +277,41 @@ class RoutedExperts(FeedForward):
             else:
                 self.shared_down.forward(act, torch.float32, out=residual, accumulate=True)
 
+    def _grouped_weights(self) -> bool:
+        """The two products of all experts can be two launches of the grouped tensor-core product."""
+        from ..kernels import gemm
+        return (self.identity == 0 and self.w_gate_up.dtype == torch.bfloat16
+                and self.w_down.dtype == torch.bfloat16 and gemm.use_tensor_cores()
+                and self.hidden_size % 8 == 0 and self.intermediate_size % 8 == 0)
+
     def _grouped(self, x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor,
-                 residual: torch.Tensor, store: bool) -> None:
+                 residual: torch.Tensor, store: bool, grouped: bool) -> None:
         from ..kernels import gemm
         n, dev = x.shape[0], x.device
         ff, width, top = self.intermediate_size, self.hidden_size, self.top
         n_pairs = n * top
-        counts = torch.zeros(self.n_outputs, dtype=torch.int32, device=dev)
         offsets = torch.empty(self.n_outputs + 1, dtype=torch.int32, device=dev)
-        order = torch.empty(n_pairs, dtype=torch.int32, device=dev)
         where = torch.empty((n, top), dtype=torch.int32, device=dev)
-        K.moe_counts(idx, counts)
-        K.moe_place(idx, counts, offsets, order, where)
         xg = torch.empty((n_pairs, width), dtype=x.dtype, device=dev)
-        K.moe_gather(x, order, xg, top)
+        if grouped and n_pairs <= GROUP_FEW_MAX:
+            K.moe_group_few(idx, x, self.n_outputs, xg, offsets, where)
+        else:
+            counts = torch.zeros(self.n_outputs, dtype=torch.int32, device=dev)
+            order = torch.empty(n_pairs, dtype=torch.int32, device=dev)
+            K.moe_counts(idx, counts)
+            K.moe_place(idx, counts, offsets, order, where)
+            K.moe_gather(x, order, xg, top)
         act = torch.empty((n_pairs, ff), dtype=x.dtype, device=dev)
         y = torch.empty((n_pairs, width), dtype=torch.float32, device=dev)
-        fused = (self.w_gate_up.dtype == torch.bfloat16 and x.dtype == torch.bfloat16
-                 and gemm.use_tensor_cores()
-                 and K.gemm_tc_supported(xg, self.w_gate_up[0]))
-        if (fused and self.identity == 0 and self.w_down.dtype == torch.bfloat16
-                and K.gemm_tc_supported(act, self.w_down[0])):
+        if grouped:
             status = gemm.status_word(dev)
             K.gemm_tc_grouped(xg, self.w_gate_up, act, offsets, status, self.activation, self.limit, self.alpha)
             K.gemm_tc_grouped(act, self.w_down, y, offsets, status)
             K.moe_combine(y, where, wts, residual, store=store)
             return
+        fused = (self.w_gate_up.dtype == torch.bfloat16 and x.dtype == torch.bfloat16
+                 and gemm.use_tensor_cores()
+                 and K.gemm_tc_supported(xg, self.w_gate_up[0]))
         first = offsets.tolist()                   # the one read of the step: rows per expert
         for e in range(self.n_outputs):
             lo, hi = first[e], first[e + 1]

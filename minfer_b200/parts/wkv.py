@@ -112,7 +112,7 @@ class Wkv(Mixer):
         K.wkv_decay(t1, self.w2t, self.w["w0"], decay)
         o = torch.empty((n, width), dtype=torch.float32, device=dev)
         K.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, self.w["u"], binding.state[WKV_STATE],
-                   ctx.cu_seqlens, ctx.slots, o, ctx.n_rows)
+                   ctx.cu_seqlens, ctx.slots, o, ctx.n_rows, ctx.max_row_tokens)
         gated = torch.empty((n, width), dtype=ctx.act_dtype, device=dev)
         K.unit_norm_gate(o, rkvg[3], 0, gated, self.n_heads, self.norm_eps, "silu",
                          weight=self.w["norm"])

@@ -92,7 +92,8 @@ def test_wkv_decay(n, rank, channels):
 # ---- the recurrences -----------------------------------------------------------------------------------
 @pytest.mark.parametrize("H,D,Dv", [(3, 12, 20), (2, 64, 64), (1, 128, 33), (5, 7, 5), (2, 160, 40), (1, 1, 1),
                                     (4, 32, 48), (1, 256, 16)])
-def test_wkv_scan_over_cuts_and_slots(H, D, Dv):
+@pytest.mark.parametrize("known", [True, False])
+def test_wkv_scan_over_cuts_and_slots(H, D, Dv, known):
     from minfer_b200.kernels import api as K
     g = torch.Generator().manual_seed(D + Dv)
     state = torch.randn(6, H, Dv, D, generator=g).to(DEV)
@@ -109,7 +110,8 @@ def test_wkv_scan_over_cuts_and_slots(H, D, Dv):
         r, k, v, d = (torch.cat([seqs[b][i][f:f + t] for b, f, t in zip(rows, first, take)]).flatten(1)
                       .contiguous().to(DEV) for i in range(4))
         out = torch.empty(r.shape[0], H * Dv, device=DEV)
-        K.wkv_scan(r, k, v, d, u.to(DEV), state, _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), out, len(rows))
+        K.wkv_scan(r, k, v, d, u.to(DEV), state, _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), out, len(rows),
+                   max(take) if known else 0)
         for i, b in enumerate(rows):
             lo = _cu(take)[i]
             got[b].append(out[lo:lo + take[i]].cpu())
@@ -123,7 +125,8 @@ def test_wkv_scan_over_cuts_and_slots(H, D, Dv):
 @pytest.mark.parametrize("H,D,Dv,cap,forget", [(3, 12, 20, 9.0, 3.0), (2, 64, 128, 15.0, 5.0), (1, 128, 31, 4.0, 0.0),
                                                (5, 7, 5, 30.0, 2.0), (2, 160, 40, 12.0, 8.0), (1, 1, 1, 1.0, 0.0),
                                                (4, 32, 15, 15.0, -6.0)])
-def test_mlstm_scan_over_cuts_and_slots(H, D, Dv, cap, forget):
+@pytest.mark.parametrize("known", [True, False])
+def test_mlstm_scan_over_cuts_and_slots(H, D, Dv, cap, forget, known):
     from minfer_b200.kernels import api as K
     g = torch.Generator().manual_seed(D * 3 + Dv)
     state = torch.randn(6, H, Dv + 1, D, generator=g).to(DEV)
@@ -151,7 +154,7 @@ def test_mlstm_scan_over_cuts_and_slots(H, D, Dv, cap, forget):
         proj[:, i_off:f_off], proj[:, f_off:f_off + H] = i, f
         out, den = torch.empty(n, H * Dv, device=DEV), torch.empty(n, H, device=DEV)
         K.mlstm_scan(proj.to(DEV), q_off, k_off, v_off, i_off, f_off, ib.to(DEV), fb.to(DEV), cap, scale, state, top,
-                     _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), out, den, len(rows))
+                     _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), out, den, len(rows), max(take) if known else 0)
         y = out.view(n, H, Dv) / den[:, :, None]
         for j, b in enumerate(rows):
             lo = _cu(take)[j]
