@@ -16,18 +16,20 @@
 // that what a lane reads of q, k and the decays from shared memory (16 bytes at a time) serves two
 // columns.  The sums of eight tokens (16 numbers a lane) are formed side by side and added over the
 // lanes by halving: each step sends what the partner keeps, 8 + 4 + 2 + 1 shuffles for all of them.  A
-// sum's tree does not depend on how the tokens are grouped.  A fifth warp does what is not the chain:
-// it keeps a ring of three chunks of tokens filled by cp.async and prepares each (wkv: r . (u k); mlstm:
-// gates and maxima), handing chunks over and taking them back through named barriers.
+// sum's tree does not depend on how the tokens are grouped.  Four more warps do what is not the
+// chain: they keep a ring of four chunks of tokens filled by cp.async, two chunks ahead, and prepare
+// each (wkv: r . (u k); mlstm: gates and maxima), handing chunks over and taking them back through
+// named barriers.
 // State [slots][heads][columns][D]: a column's elements are contiguous.  Every column keeps its own
 // copy of the running maximum ([slots][heads][columns]), so no block reads what another writes.
 // Tokens are packed row after row (row b: tokens cu_seqlens[b] .. cu_seqlens[b + 1]).
 #include "common.cuh"
 
-#define OS_THREADS 128       // the threads that walk the tokens; one more warp feeds them
+#define OS_THREADS 128       // the threads that walk the tokens
+#define OS_FEED 4            // warps that feed them
 #define OS_TU 8              // tokens whose sums are formed side by side
 #define OS_TC 16             // tokens of a chunk
-#define OS_STAGES 3
+#define OS_STAGES 4
 #define OS_MAX_D 256
 
 struct OuterScanArgs {
@@ -79,12 +81,12 @@ __device__ __forceinline__ void os_reduce16(float (&a)[16], int l) {
     if (LD == 32) a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
 }
 
-// named barriers of the hand-over (0 is __syncthreads): all five warps take part
+// named barriers of the hand-over (0 is __syncthreads): all eight warps take part
 __device__ __forceinline__ void os_bar_sync(int id) {
-    asm volatile("bar.sync %0, %1;" ::"r"(id), "n"(OS_THREADS + 32) : "memory");
+    asm volatile("bar.sync %0, %1;" ::"r"(id), "n"(OS_THREADS + 32 * OS_FEED) : "memory");
 }
 __device__ __forceinline__ void os_bar_arrive(int id) {
-    asm volatile("bar.arrive %0, %1;" ::"r"(id), "n"(OS_THREADS + 32) : "memory");
+    asm volatile("bar.arrive %0, %1;" ::"r"(id), "n"(OS_THREADS + 32 * OS_FEED) : "memory");
 }
 #define OS_FULL(stage) (1 + (stage))
 #define OS_EMPTY(stage) (1 + OS_STAGES + (stage))
@@ -128,7 +130,7 @@ __device__ __forceinline__ float os_soft_cap(float z, float cap) { return cap * 
 // LD: lanes that share a pair of columns; ND4: float4 groups of a column a lane holds (D <= 4 LD ND4);
 // tc: tokens of a chunk
 template <int LD, int ND4, bool WKV>
-__global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanArgs a, int tc) {
+__global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(OuterScanArgs a, int tc) {
     pdl_launch_dependents();
     constexpr int DP = 4 * LD * ND4;                   // padded key size
     constexpr int TV = 2 * (OS_THREADS / LD);          // columns of a block
@@ -148,14 +150,15 @@ __global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanAr
     const int n_chunks = (n_b + tc - 1) / tc;
     if (n_b <= 0) { pdl_wait(); return; }
 
-    if (warp == OS_THREADS / 32) {
-        // ---- the feeding warp ----------------------------------------------------------------------
+    if (warp >= OS_THREADS / 32) {
+        // ---- the feeding warps: each takes every OS_FEED-th token of a chunk, the first the gates too ----------------------------------------------------------------------
         // (a row of a tensor may start anywhere: 16-byte copies only where all of them start on 16 bytes)
         const bool vec = (D & 3) == 0 &&
                          ((a.r_width | a.k_width | a.w_width | (long long)(a.r_off | a.k_off | a.w_off)) & 3) == 0 &&
                          (((uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.w) & 15) == 0;
         const bool vec_v = (Dv & 3) == 0 && ((a.v_width | (long long)a.v_off) & 3) == 0 && ((uintptr_t)a.v & 15) == 0;
-        if (DP > D) {                                  // the copies never touch the padding
+        const int fw = warp - OS_THREADS / 32;
+        if (DP > D && fw == 0) {                       // the copies never touch the padding
             const int pad = DP - D;
             for (int i = lane; i < OS_STAGES * tc * NVEC * pad; i += 32) {
                 const int row = i / pad, d = D + i - row * pad;
@@ -168,7 +171,12 @@ __global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanAr
         pdl_wait();
         float m_run = 0.f;
         if (!WKV) m_run = a.maxima[((size_t)slot * a.heads + h) * cols + j0];
-        float next_i = 0.f, next_f = 0.f;              // raw gates of the chunk asked for last
+        float raw_i[3] = {0.f, 0.f, 0.f}, raw_f[3] = {0.f, 0.f, 0.f};   // raw gates: this chunk's, the next two's
+        float bonus[DP / 32];                          // (wkv) this lane's share of the head's bonus
+        if (WKV) {
+#pragma unroll
+            for (int e = 0; e < DP / 32; ++e) bonus[e] = lane + 32 * e < D ? a.u[h * D + lane + 32 * e] : 0.f;
+        }
         const int v_cols = min(n_cols, Dv - j0);       // columns of the tile that have values (may be 0)
         auto fetch = [&](int chunk) {
             const int c0 = chunk * tc, nc = min(tc, n_b - c0);
@@ -181,7 +189,9 @@ __global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanAr
             const float* kg = a.k + t * a.k_width + a.k_off + h * D;
             const float* wg = WKV ? a.w + t * a.w_width + a.w_off + h * D : nullptr;
             const float* vg = a.v + t * a.v_width + a.v_off + (size_t)h * Dv + j0;
-            for (int tt = 0; tt < nc; ++tt) {
+            r_s += fw * DP; k_s += fw * DP; w_s += fw * DP;
+            rg += fw * a.r_width; kg += fw * a.k_width; if (WKV) wg += fw * a.w_width;
+            for (int tt = fw; tt < nc; tt += OS_FEED) {
                 if (vec) {
                     for (int d = 4 * lane; d < D; d += 128) {
                         os_cp16(r_s + d, rg + d);
@@ -195,65 +205,88 @@ __global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanAr
                         if (WKV) os_cp4(w_s + d, wg + d);
                     }
                 }
-                r_s += DP; k_s += DP; w_s += DP;
-                rg += a.r_width; kg += a.k_width; if (WKV) wg += a.w_width;
+                r_s += OS_FEED * DP; k_s += OS_FEED * DP; w_s += OS_FEED * DP;
+                rg += OS_FEED * a.r_width; kg += OS_FEED * a.k_width; if (WKV) wg += OS_FEED * a.w_width;
             }
             if (vec_v && (v_cols & 3) == 0) {
                 const int per = v_cols >> 2;
-                for (int i = lane; i < nc * per; i += 32) {
+                for (int i = 32 * fw + lane; i < nc * per; i += 32 * OS_FEED) {
                     const int tt = i / per, cc = (i - tt * per) << 2;
                     os_cp16(v_s + tt * TV + cc, vg + (size_t)tt * a.v_width + cc);
                 }
             } else {
-                for (int i = lane; i < nc * v_cols; i += 32) {
+                for (int i = 32 * fw + lane; i < nc * v_cols; i += 32 * OS_FEED) {
                     const int tt = i / v_cols, cc = i - tt * v_cols;
                     os_cp4(v_s + tt * TV + cc, vg + (size_t)tt * a.v_width + cc);
                 }
             }
-            if (!WKV) {
+            if (!WKV && fw == 0) {
                 if (j0 + n_cols == cols)               // the normalizer's column
                     for (int tt = lane; tt < nc; tt += 32) v_s[tt * TV + n_cols - 1] = 1.0f;
+                raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1];
+                raw_i[1] = raw_i[2]; raw_f[1] = raw_f[2];
                 if (lane < nc) {
                     const float* g = a.gates + (t + lane) * a.gate_width + h;
-                    next_i = g[a.i_off];
-                    next_f = g[a.f_off];
+                    raw_i[2] = g[a.i_off];
+                    raw_f[2] = g[a.f_off];
                 }
             }
         };
-        fetch(0);
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        // two chunks ahead; a chunk that does not exist is an empty group of copies
+        for (int ahead = 0; ahead < 2; ++ahead) {
+            if (ahead < n_chunks) fetch(ahead);
+            else if (!WKV) { raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1]; raw_i[1] = raw_i[2]; raw_f[1] = raw_f[2]; }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        }
         for (int chunk = 0; chunk < n_chunks; ++chunk) {
             const int nc = min(tc, n_b - chunk * tc);
-            const float raw_i = next_i, raw_f = next_f;
-            if (chunk + 1 < n_chunks) {
-                if (chunk + 1 >= OS_STAGES) os_bar_sync(OS_EMPTY((chunk + 1) % OS_STAGES));
-                fetch(chunk + 1);
+            if (chunk + 2 < n_chunks) {
+                if (chunk + 2 >= OS_STAGES) os_bar_sync(OS_EMPTY((chunk + 2) % OS_STAGES));
+                fetch(chunk + 2);
+            } else if (!WKV) {
+                raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1];
+                raw_i[1] = raw_i[2]; raw_f[1] = raw_f[2];
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
+            asm volatile("cp.async.wait_group 2;" ::: "memory");
             __syncwarp();                              // every lane's copies of this chunk are there
             float* r_s = os_smem + (chunk % OS_STAGES) * stage_floats;
             float* k_s = r_s + tc * DP;
             float* f_s = r_s + tc * (NVEC * DP + TV);
             if (WKV) {
-                // r . (u k): what the current token's own value is multiplied by
-                float s[16];
+                // r . (u k), of the tokens this warp copied: what the current token's own value is
+                // multiplied by
+                constexpr int OWN = OS_TC / OS_FEED;
+                float s[OWN];
 #pragma unroll
-                for (int tt = 0; tt < 16; ++tt) s[tt] = 0.f;
-                for (int d = lane; d < D; d += 32) {
-                    const float ud = a.u[h * D + d];
+                for (int i = 0; i < OWN; ++i) s[i] = 0.f;
 #pragma unroll
-                    for (int tt = 0; tt < 16; ++tt)
-                        if (tt < nc) s[tt] = fmaf(r_s[tt * DP + d] * ud, k_s[tt * DP + d], s[tt]);
+                for (int e = 0; e < DP / 32; ++e) {
+                    const int d = lane + 32 * e;
+                    if (d < D) {
+#pragma unroll
+                        for (int i = 0; i < OWN; ++i) {
+                            const int tt = fw + OS_FEED * i;
+                            if (tt < nc) s[i] = fmaf(r_s[tt * DP + d] * bonus[e], k_s[tt * DP + d], s[i]);
+                        }
+                    }
                 }
-                os_reduce16<32>(s, lane);
-                if ((lane & 1) == 0 && (lane >> 1) < nc) f_s[lane >> 1] = s[0];
-            } else {
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+#pragma unroll
+                    for (int i = 0; i < OWN; ++i) s[i] += __shfl_xor_sync(0xffffffffu, s[i], o);
+                }
+                if (lane == 0) {
+#pragma unroll
+                    for (int i = 0; i < OWN; ++i)
+                        if (fw + OS_FEED * i < nc) f_s[fw + OS_FEED * i] = s[i];
+                }
+            } else if (fw == 0) {
                 // a token a lane; the maxima by a scan in which a stretch of tokens is the pair
                 // (sum of f, largest i + the f's after it)
                 const bool mine = lane < nc;
-                const float li = mine ? os_soft_cap(raw_i + ib, a.cap) : -INFINITY;
-                const float zf = mine ? os_soft_cap(raw_f + fb, a.cap) : 0.f;
+                const float li = mine ? os_soft_cap(raw_i[0] + ib, a.cap) : -INFINITY;
+                const float zf = mine ? os_soft_cap(raw_f[0] + fb, a.cap) : 0.f;
                 const float lf = mine ? fminf(zf, 0.f) - log1pf(expf(-fabsf(zf))) : 0.f;
                 float F = lf, M = li;
 #pragma unroll
@@ -275,7 +308,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32) outer_scan_kernel(OuterScanAr
             }
             os_bar_arrive(OS_FULL(chunk % OS_STAGES));
         }
-        if (!WKV)
+        if (!WKV && fw == 0)
             for (int i = lane; i < n_cols; i += 32) a.maxima[((size_t)slot * a.heads + h) * cols + j0 + i] = m_run;
         return;
     }
@@ -408,7 +441,7 @@ static int os_launch(const OuterScanArgs& a, int max_tokens, cudaStream_t stream
     }
     const int cols = WKV ? a.Dv : a.Dv + 1;
     const int tiles = (cols + TV - 1) / TV;
-    mf_launch(outer_scan_kernel<LD, ND4, WKV>, dim3(a.heads * tiles, a.n_rows), dim3(OS_THREADS + 32), bytes(tc),
+    mf_launch(outer_scan_kernel<LD, ND4, WKV>, dim3(a.heads * tiles, a.n_rows), dim3(OS_THREADS + 32 * OS_FEED), bytes(tc),
               stream, a, tc);
     return MF_LAUNCH_CHECK();
 }
