@@ -90,10 +90,12 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_decode_kernel(LatentArgs
         if (page < 0) page = 0;                       // (masked: no visible position lies there)
         const __nv_bfloat16* src = a.k + (size_t)page * MF_PAGE * a.kw;
         const uint32_t dst = k_base + (uint32_t)(buf * MF_PAGE * pitch);
-        for (int i = tid; i < MF_PAGE * chunks; i += LA_WARPS * 32) {
-            const int r = i / chunks, c = i - r * chunks;
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;"
-                         ::"r"(dst + (uint32_t)(r * pitch + c * 16)), "l"(src + (size_t)i * 8) : "memory");
+#pragma unroll
+        for (int i = 0; i < MF_PAGE / LA_WARPS; ++i) {
+            const int r = warp + LA_WARPS * i;
+            for (int c = lane; c < chunks; c += 32)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;"
+                             ::"r"(dst + (uint32_t)(r * pitch + c * 16)), "l"(src + (size_t)r * a.kw + c * 8) : "memory");
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -250,19 +252,24 @@ latent_combine_kernel(const float* __restrict__ partial, __nv_bfloat16* __restri
     m = block_max(m, scratch);
     float l = 0.f;
     for (int c = threadIdx.x; c < n_splits; c += blockDim.x) {
-        const float f = exp2f(p[c * stride] - m);      // (a split that saw nothing has maximum -inf: 0)
+        const float2 ml = *reinterpret_cast<const float2*>(p + c * stride);
+        const float f = exp2f(ml.x - m);               // (a split that saw nothing has maximum -inf: 0)
         f_s[c] = f;
-        l = fmaf(p[c * stride + 1], f, l);
+        l = fmaf(ml.y, f, l);
     }
     l = block_sum(l, scratch);                         // (its barriers also publish f_s)
     if (sink) l += exp2f(sink2 - m);
     const float inv = 1.0f / l;
-    for (int d = threadIdx.x; d < vd; d += blockDim.x) {
+    for (int d = 2 * threadIdx.x; d < vd; d += 2 * blockDim.x) {
         const float* pd = p + 2 + d;
-        float acc = 0.f;
-#pragma unroll 8
-        for (int c = 0; c < n_splits; ++c) acc = fmaf(pd[c * stride], f_s[c], acc);
-        out[rh * vd + d] = __float2bfloat16_rn(acc * inv);
+        float2 acc = make_float2(0.f, 0.f);
+#pragma unroll 16
+        for (int c = 0; c < n_splits; ++c) {
+            const float2 x = *reinterpret_cast<const float2*>(pd + c * stride);
+            acc.x = fmaf(x.x, f_s[c], acc.x);
+            acc.y = fmaf(x.y, f_s[c], acc.y);
+        }
+        *reinterpret_cast<__nv_bfloat162*>(out + rh * vd + d) = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
     }
 }
 
@@ -332,7 +339,7 @@ extern "C" int mf_latent_decode(const void* q, const void* k_cache, const int* r
     else if (vd <= 512) e = la_launch<4>(a, rows, stream);
     else e = la_launch<5>(a, rows, stream);
     if (e || a.n_splits == 1) return e;
-    mf_launch_ex(false, latent_combine_kernel, dim3(rows * n_heads), dim3(vd <= 128 ? 128 : 256), 0, stream, (const float*)partial,
+    mf_launch_ex(false, latent_combine_kernel, dim3(rows * n_heads), dim3(vd <= 256 ? 128 : 256), 0, stream, (const float*)partial,
                  (__nv_bfloat16*)out, a.n_splits, vd, a.sink, sink_logit, n_heads);
     return MF_LAUNCH_CHECK();
 }

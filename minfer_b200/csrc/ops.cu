@@ -1547,7 +1547,7 @@ __device__ __forceinline__ void term_value(const ScaledTerm& s, size_t at, size_
 #pragma unroll
     for (int j = 0; j < VEC; ++j) v[j] = 0.0f;
     if (s.y) RowVec<float, VEC>::load(s.y + at, v);
-#pragma unroll 4
+#pragma unroll 8
     for (int p = 0; p < s.n_part; ++p) {
         float q[VEC];
         RowVec<float, VEC>::load(s.part + (size_t)p * split + at, q);

@@ -494,7 +494,7 @@ wkv_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* 
     int r = 0;
     // four numbers of the rank at a time (every row of wd_s starts on 16 bytes); few tokens: more of the
     // matrix's loads in flight, since nothing else hides them
-    constexpr int AHEAD = NT <= 2 ? 4 : 1;
+    constexpr int AHEAD = NT <= 2 ? 4 : 2;
     for (; r + 4 * AHEAD <= rank; r += 4 * AHEAD) {
         float w[4 * AHEAD];
 #pragma unroll
