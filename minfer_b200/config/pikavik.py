@@ -1,9 +1,9 @@
 """Typed configuration of the Pikavik decoder, read from its own config.json keys.
 
 The design: token embedding; layers with one norm that both sublayers read, x += a1 * mixer(y) +
-a2 * ff(y) with learned vectors a1 and a2 (the feed-forward optional); every norm weight of the stream
-is stored around zero (1 + w).  The mixer is RWKV-style time mixing, the matrix memory of xLSTM, or
-latent attention whose queries go through a latent too (rotated part shared by all heads, a learned
+a2 * ff(y) with learned vectors a1 and a2 (the feed-forward optional); the
+norms of the stream multiply by 1 + w.  The mixer is WKV, mLSTM, or latent
+attention whose queries go through a latent too (rotated part shared by all heads, a learned
 sink per head); the feed-forward is routed (sigmoid scores, experts chosen within the best groups, a
 clamped activation, a gated shared expert).  Final norm, head.  config.json keys:
 

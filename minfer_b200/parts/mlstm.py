@@ -1,5 +1,5 @@
-"""The matrix memory of xLSTM as a mixer: a state per head that exponential gates fill and empty, kept
-in range by a running maximum, with a normalizer.
+"""mLSTM as a mixer: a matrix-valued state per head that exponential gates fill and empty, kept in range
+by a running maximum, with a normalizer.
 
     q = Wq u * head_dim^(-1/2),  k = Wk u  (heads of ``head_dim``),  v = Wv u  (heads of ``value_dim``)
     per head  i = cap tanh((Wi u + bi) / cap),  f = log sigmoid(cap tanh((Wf u + bf) / cap))

@@ -2,7 +2,7 @@
 (src/vec_ops.rs:500-522; src/graph/cpu_backend.rs:195-213).
 
 Three options for architectures that want them: ``offset`` (a constant added to the stored weight: a
-checkpoint that stores its norm weights around zero has offset 1), ``tensor_name`` (the weight's whole name behind
+checkpoint that holds its norm weights as differences from 1 has offset 1), ``tensor_name`` (the weight's whole name behind
 the prefix, for checkpoints that do not call it ``<name>.weight``) and ``gain`` (a constant
 factor on the output, y = x / rms * w * gain, held as w * gain: a model's logit scale rides
 on its last norm this way at no cost)."""

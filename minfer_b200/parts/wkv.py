@@ -1,4 +1,4 @@
-"""RWKV-style time mixing as a mixer: linear attention with a data-dependent decay per key channel, a
+"""WKV, the recurrence of the RWKV models, as a mixer: linear attention with a data-dependent decay per key channel, a
 bonus for the current token, and inputs that are each mixed with the token before.
 
     u' = the u of the sequence's token before (zeros for the first)

@@ -379,3 +379,44 @@ def test_latent_decode_every_token_of_a_portion_is_a_query():
         k = keys[0][:p + 1].double()
         want = torch.softmax(torch.einsum("hd,jd->hj", q[0][i].double(), k) * 0.1, dim=-1) @ k[:, :vd]
         _close(out[i], want, 1.5e-2)
+
+
+# ---- few tokens ------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("n,top,experts,width", [(1, 1, 1, 8), (5, 3, 7, 64), (48, 4, 16, 100), (200, 5, 40, 24)])
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16])
+def test_group_few(n, top, experts, width, dt):
+    """Pairs grouped by expert in their order, the experts' first rows (also of experts nobody chose)
+    and the gathered inputs."""
+    from minfer_b200.kernels import api as K
+    if width * (4 if dt == torch.float32 else 2) % 16:
+        width += 4
+    g = torch.Generator().manual_seed(n)
+    idx = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(n)]).int()
+    x = torch.randn(n, width, generator=g).to(dt)
+    out = torch.empty(n * top, width, dtype=dt, device=DEV)
+    first, where = torch.empty(experts + 1, dtype=torch.int32, device=DEV), torch.empty(n, top, dtype=torch.int32, device=DEV)
+    K.moe_group_few(idx.to(DEV), x.to(DEV), experts, out, first, where)
+    order = torch.argsort(idx.flatten().long(), stable=True)
+    rows = torch.empty_like(order)
+    rows[order] = torch.arange(n * top)
+    assert torch.equal(where.cpu().flatten().long(), rows)
+    assert first.tolist() == [int((idx < e).sum()) for e in range(experts + 1)]
+    assert torch.equal(out.cpu(), x[order // top])
+
+
+@pytest.mark.parametrize("n", [1, 7, 8, 16, 17])
+@pytest.mark.parametrize("heads,J,D,tail,gated", [(3, 40, 24, 16, False), (16, 24, 264, 0, True), (1, 5, 8, 8, False)])
+def test_per_head_products_of_few_tokens(n, heads, J, D, tail, gated):
+    from minfer_b200.kernels import api as K
+    g = torch.Generator().manual_seed(n + J)
+    x = torch.randn(n, heads * (D + tail), generator=g).bfloat16()
+    w = (torch.randn(heads, J, D, generator=g) * D ** -0.5).bfloat16()
+    gate = torch.randn(n, 3 + heads * J, generator=g)
+    y = torch.empty(n, heads * (J + tail), dtype=torch.bfloat16, device=DEV)
+    K.head_linear(x.to(DEV), w.to(DEV), y, x_head=D + tail, x_off=0, y_head=J + tail, tail=tail, x_tail_off=D,
+                  gate=gate.to(DEV) if gated else None, gate_off=3)
+    xh = x.double().view(n, heads, D + tail)
+    want = torch.einsum("hjd,nhd->nhj", w.double(), xh[..., :D])
+    if gated:
+        want = want * torch.sigmoid(gate.double()[:, 3:].view(n, heads, J))
+    _close(y.view(n, heads, J + tail), torch.cat([want, xh[..., D:]], dim=-1), 6e-3)
