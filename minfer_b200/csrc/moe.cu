@@ -181,9 +181,9 @@ extern "C" int mf_moe_route_scored(const float* logits, long long stride, const 
     return MF_LAUNCH_CHECK();
 }
 
-// Scores = sigmoid of each router output.  The experts form `groups` equal groups of neighbours; a
-// group's score is the sum of its two largest scores, and only experts of the `keep` best groups can
-// be chosen (groups 1: all).  The `top` largest scores among them are chosen (ties anywhere: the
+// Scores = sigmoid of each router output.  The experts are cut into `groups` runs of
+// equal length, ranked by their two best scores added up; the choice is among the experts of the `keep`
+// first-ranked runs (groups 1: among all).  The `top` largest scores among them are chosen (ties anywhere: the
 // lower index), with weights score / (sum of the chosen scores + 1e-20) * scale.  A warp per token.
 __global__ void __launch_bounds__(256)
 moe_route_groups_kernel(const float* __restrict__ logits, long long stride, int* __restrict__ idx,

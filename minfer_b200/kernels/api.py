@@ -1320,8 +1320,8 @@ def moe_route_scored(logits: torch.Tensor, correction: Optional[torch.Tensor], i
 def moe_route_groups(logits: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, top: int, outputs: int,
                      groups: int = 1, keep: int = 1, scale: float = 1.0) -> None:
     """Per row of ``logits`` (float32 [tokens, >= outputs]; only the first ``outputs`` columns are the
-    router's): scores = sigmoid; the outputs form ``groups`` equal groups of neighbours, a group's
-    score is the sum of its two largest, and the ``top`` largest scores within the ``keep`` best
+    router's): scores = sigmoid; the outputs are cut into ``groups`` runs of equal length,
+    ranked by the two best scores of each added up; the ``top`` largest scores within the ``keep`` best
     groups (ties: the lower index) go into ``idx``, score / (sum of the chosen + 1e-20) * ``scale``
     into ``wts``."""
     n = logits.shape[0]

@@ -12,8 +12,8 @@ Options for designs that route otherwise (each a parameter):
                             largest s + correction are chosen (``correction_name``: a tensor of one
                             number per output; None: none); the weights are the chosen s themselves,
                             not renormalized
-    scoring "sigmoid_groups" scores s = sigmoid(z); the experts form ``groups`` equal groups of neighbours,
-                            a group's score is the sum of its two largest s, and the ``top`` largest s
+    scoring "sigmoid_groups" scores s = sigmoid(z); the experts are cut into ``groups`` runs of equal
+                            length, ranked by the two best s of each added up; the ``top`` largest s
                             within the ``keep_groups`` best groups are chosen; their weights are
                             s / (sum of the chosen s + 1e-20) * ``weight_scale``
     identity                the last ``identity`` router outputs (beyond the ``n_experts`` experts with
