@@ -55,8 +55,9 @@
 #define EPI_GATE_GELU_TANH 1
 #define EPI_GATE_CLAMPED_SWISH 2   // g' sigmoid(act_n g') (u' + 1), g' = min(g, act_p), u' = clamp(u, -act_p, act_p)
 #define EPI_PARTIAL 3         // ws[split][token][n] = acc (float32)
-#define EPI_XIELU 4           // out = f(acc + bias), f(z) = act_p z^2 + z/2 (z > 0),
-                              // act_n (exp(z) - 1 - z) + z/2 (z <= 0)   (float32 or bfloat16)
+#define EPI_XIELU 4           // out = f(acc + bias), f(z) = act_p z^2 + act_l z (z > 0),
+                              // act_n (exp(z) - 1 - z) + act_l z (z <= 0)   (float32 or bfloat16):
+                              // xIELU (act_l = 1/2) and, with act_p = 1 and the others 0, relu squared
 
 #define MF_ERR_NO_TENSORMAP 2003
 #define MF_ERR_TENSORMAP 2004
@@ -82,7 +83,7 @@ struct GemmArgs {
     const float* prep_g;
     float* prep_ssq;
     long long ldp;            // elements between consecutive tokens of prep_x
-    float act_p, act_n;       // EPI_XIELU: the two coefficients of the activation
+    float act_p, act_n, act_l;   // EPI_XIELU: the activation's coefficients
     int gate_act;             // EPI_SWIGLU: 0 silu, EPI_GATE_GELU_TANH
     // grouped products: group g's token rows are group_first[g] .. group_first[g + 1] (device memory)
     // or, with group_first null, g * group_rows .. (g + 1) * group_rows; its weight rows g * N ..
@@ -281,8 +282,8 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& a, const uint32_t* r
         for (int jj = 0; jj < 8; ++jj) {
             float v0 = __uint_as_float(r[2 * jj]) + bias, v1 = __uint_as_float(r[2 * jj + 1]) + bias;
             if (a.epi == EPI_XIELU) {
-                v0 = v0 > 0.0f ? fmaf(a.act_p * v0, v0, 0.5f * v0) : fmaf(a.act_n, (__expf(v0) - 1.0f) - v0, 0.5f * v0);
-                v1 = v1 > 0.0f ? fmaf(a.act_p * v1, v1, 0.5f * v1) : fmaf(a.act_n, (__expf(v1) - 1.0f) - v1, 0.5f * v1);
+                v0 = v0 > 0.0f ? fmaf(a.act_p * v0, v0, a.act_l * v0) : fmaf(a.act_n, (__expf(v0) - 1.0f) - v0, a.act_l * v0);
+                v1 = v1 > 0.0f ? fmaf(a.act_p * v1, v1, a.act_l * v1) : fmaf(a.act_n, (__expf(v1) - 1.0f) - v1, a.act_l * v1);
             }
             const float keep = even ? v0 : v1, send = even ? v1 : v0;
             const float recv = __shfl_xor_sync(0xffffffffu, send, 1);
@@ -298,8 +299,8 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& a, const uint32_t* r
             const int tok = tok0 + j;
             float v = __uint_as_float(r[j]) + bias;
             if (a.epi == EPI_XIELU)
-                v = v > 0.0f ? fmaf(a.act_p * v, v, 0.5f * v)
-                             : fmaf(a.act_n, (__expf(v) - 1.0f) - v, 0.5f * v);
+                v = v > 0.0f ? fmaf(a.act_p * v, v, a.act_l * v)
+                             : fmaf(a.act_n, (__expf(v) - 1.0f) - v, a.act_l * v);
             if (tok < a.M && n_ok) {
                 if (a.epi == EPI_PARTIAL)
                     a.partial[((size_t)split * a.M + tok) * a.N + n] = v;
@@ -1306,7 +1307,7 @@ struct FusedNorm {
     long long ldp;
     const float* prep_g;      // ... its weight [N] ...
     float* prep_ssq;          // ... and the sums of squares [parts][M] this product writes
-    float act_p = 0.0f, act_n = 0.0f;   // EPI_XIELU
+    float act_p = 0.0f, act_n = 0.0f, act_l = 0.0f;   // EPI_XIELU
 };
 
 
@@ -1366,7 +1367,7 @@ static int gemm_tc_impl(const void* x, long long ldx, const void* w, long long l
     if (f != nullptr) {
         a.row_ssq = f->row_ssq; a.ssq_parts = f->ssq_parts; a.ssq_width = f->ssq_width; a.ssq_eps = f->ssq_eps;
         a.prep_x = f->prep_x; a.ldp = f->ldp; a.prep_g = f->prep_g; a.prep_ssq = f->prep_ssq;
-        a.act_p = f->act_p; a.act_n = f->act_n;
+        a.act_p = f->act_p; a.act_n = f->act_n; a.act_l = f->act_l;
     }
     if (pair_mode_on() && M >= 256 && splits == 1) {
         if (a.row_ssq != nullptr) return MF_ERR_UNSUPPORTED;     // the CTA-pair kernel applies no row scale
@@ -1467,18 +1468,18 @@ extern "C" int mf_gemm_tc_fused(const void* x, long long ldx, const void* w, lon
                         status, &f, stream);
 }
 
-// out = f(x w^T) with the xIELU activation f(z) = act_p z^2 + z/2 (z > 0), act_n (exp(z) - 1 - z)
-// + z/2 (z <= 0) applied to the float32 sums in the epilogue (never split along K); `row_ssq`
+// out = f(x w^T) with the activation f(z) = act_p z^2 + act_l z (z > 0), act_n (exp(z) - 1 - z)
+// + act_l z (z <= 0) applied to the float32 sums in the epilogue (never split along K); `row_ssq`
 // as in mf_gemm_tc_fused.
 extern "C" int mf_gemm_tc_xielu(const void* x, long long ldx, const void* w, long long ldw,
                                 void* out, long long ldo, int out_dtype, int M, int N, int K,
-                                float act_p, float act_n, const float* row_ssq, int ssq_parts,
+                                float act_p, float act_n, float act_l, const float* row_ssq, int ssq_parts,
                                 int ssq_width, float ssq_eps, unsigned* status,
                                 cudaStream_t stream) {
     FusedNorm f;
     f.row_ssq = row_ssq; f.ssq_parts = ssq_parts; f.ssq_width = ssq_width; f.ssq_eps = ssq_eps;
     f.prep_x = nullptr; f.ldp = 0; f.prep_g = nullptr; f.prep_ssq = nullptr;
-    f.act_p = act_p; f.act_n = act_n;
+    f.act_p = act_p; f.act_n = act_n; f.act_l = act_l;
     return gemm_tc_impl(x, ldx, w, ldw, nullptr, out, ldo, out_dtype, M, N, K, EPI_XIELU, nullptr,
                         nullptr, status, &f, stream);
 }

@@ -1261,7 +1261,7 @@ extern "C" int mf_norm_add(float* h, const float* base, const float* partial, in
 
 // ------------------------------------------------------------------------------------
 // Activations on float32 products, written in the activation type.
-//   unary_act    kind 0: the erf form of gelu, 0.5 z (1 + erf(z / sqrt 2))
+//   unary_act    kind 0: the erf form of gelu, 0.5 z (1 + erf(z / sqrt 2)); kind 1: max(z, 0)^2
 //   row_gate_mul o[t][:] <- o[t][:] * sigmoid(gate[t * gate_stride]), in place: one number a row
 //   gated_act    from rows [gate (ff) | up (ff)] (or, interleaved, gate, up, gate, up, ..): kind 0 silu(g) u; kind 1 gelu_tanh(g) u;
 //                kind 2 the clamped form g' sigmoid(alpha g') (u' + 1), g' = min(g, limit),
@@ -1281,7 +1281,8 @@ __global__ void unary_act_kernel(const float* __restrict__ z, TO* __restrict__ o
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n;
          i += (long long)gridDim.x * blockDim.x) {
         const float v = z[i];
-        out[i] = from_f32<TO>(0.5f * v * (1.0f + erff(v * 0.7071067811865476f)));
+        const float p = fmaxf(v, 0.0f);
+        out[i] = from_f32<TO>(kind == 1 ? p * p : 0.5f * v * (1.0f + erff(v * 0.7071067811865476f)));
     }
 }
 
@@ -1294,7 +1295,7 @@ static inline dim3 mf_flat_grid(long long n) {
 extern "C" int mf_unary_act(const float* z, void* out, int out_dtype, long long n, int kind,
                             cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (kind != 0) return MF_ERR_ARGUMENT;
+    if (kind != 0 && kind != 1) return MF_ERR_ARGUMENT;
     if (out_dtype == MF_DTYPE_F32)
         mf_launch(unary_act_kernel<float>, mf_flat_grid(n), dim3(256), 0, stream, z, (float*)out, n, kind);
     else if (out_dtype == MF_DTYPE_BF16)
@@ -1631,5 +1632,155 @@ extern "C" int mf_scaled_add(float* h, const float* y1, const float* part1, int 
     else if (out_dtype == MF_DTYPE_BF16) { if (vec) MF_SA(__nv_bfloat16, 4); else MF_SA(__nv_bfloat16, 1); }
     else return MF_ERR_UNSUPPORTED;
 #undef MF_SA
+    return MF_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------
+// norm_terms: the end of a sublayer whose OUTPUT is normed before it joins the stream, with the norm
+// that reads the stream next.  With T_k the k-th term (`y` plus the K splits `part` of a product, as in
+// scaled_add) and rms over a row of `width` numbers, eps inside the root:
+//     v = mult * (T_1 / rms(T_1) * w_1 [+ T_2 / rms(T_2) * w_2])          (a term's `scale` is w_k)
+//     v <- v / rms(v) * out_w                                             (out_w null: left out)
+//     h += v;   x_out = h / rms(h) * next_w                               (x_out null: left out)
+// A block per row, the row in registers (width up to 4 * VEC * blockDim).
+// ------------------------------------------------------------------------------------
+struct NormTermsArgs {
+    float* h;
+    ScaledTerm t1, t2;
+    const float* out_w;
+    const float* next_w;
+    void* x_out;
+    int width;
+    float mult, eps, out_eps, next_eps;
+};
+
+// the sums of two numbers over a block (as block_sum for each)
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* scratch) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        a += __shfl_xor_sync(0xffffffffu, a, o);
+        b += __shfl_xor_sync(0xffffffffu, b, o);
+    }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n = blockDim.x >> 5;
+    if (lane == 0) scratch[warp] = make_float2(a, b);
+    __syncthreads();
+    float2 v = lane < n ? scratch[lane] : make_float2(0.f, 0.f);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        v.x += __shfl_xor_sync(0xffffffffu, v.x, o);
+        v.y += __shfl_xor_sync(0xffffffffu, v.y, o);
+    }
+    return v;
+}
+
+template <typename TO, int VEC, bool PAIR>
+__global__ void __launch_bounds__(1024) norm_terms_kernel(NormTermsArgs a) {
+    pdl_launch_dependents();
+    __shared__ float2 scratch[3][32];
+    const int width = a.width;
+    const size_t base = (size_t)blockIdx.x * width, split = (size_t)gridDim.x * width;
+    pdl_wait();
+    float u[4][VEC], g[PAIR ? 4 : 1][VEC];
+    float s1 = 0.0f, s2 = 0.0f;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int i = (threadIdx.x + r * blockDim.x) * VEC;
+        if (i < width) {
+            term_value<VEC>(a.t1, base + i, split, u[r]);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) s1 = fmaf(u[r][j], u[r][j], s1);
+            if (PAIR) {
+                term_value<VEC>(a.t2, base + i, split, g[PAIR ? r : 0]);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) s2 = fmaf(g[PAIR ? r : 0][j], g[PAIR ? r : 0][j], s2);
+            }
+        }
+    }
+    float2 ss = block_sum2(s1, s2, scratch[0]);
+    const float f1 = a.mult / sqrtf(ss.x / (float)width + a.eps);
+    const float f2 = PAIR ? a.mult / sqrtf(ss.y / (float)width + a.eps) : 0.0f;
+    s1 = 0.0f;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int i = (threadIdx.x + r * blockDim.x) * VEC;
+        if (i < width) {
+            float w[VEC];
+            RowVec<float, VEC>::load(a.t1.scale + i, w);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) u[r][j] *= f1 * w[j];
+            if (PAIR) {
+                RowVec<float, VEC>::load(a.t2.scale + i, w);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) u[r][j] = fmaf(g[PAIR ? r : 0][j], f2 * w[j], u[r][j]);
+            }
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) s1 = fmaf(u[r][j], u[r][j], s1);
+        }
+    }
+    float fo = 1.0f;
+    if (a.out_w) {
+        ss = block_sum2(s1, 0.0f, scratch[1]);
+        fo = 1.0f / sqrtf(ss.x / (float)width + a.out_eps);
+    }
+    s1 = 0.0f;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int i = (threadIdx.x + r * blockDim.x) * VEC;
+        if (i < width) {
+            float h[VEC];
+            RowVec<float, VEC>::load(a.h + base + i, h);
+            if (a.out_w) {
+                float w[VEC];
+                RowVec<float, VEC>::load(a.out_w + i, w);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) u[r][j] *= fo * w[j];
+            }
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                u[r][j] += h[j];
+                s1 = fmaf(u[r][j], u[r][j], s1);
+            }
+            row_store<float, VEC>(a.h + base + i, u[r]);
+        }
+    }
+    if (a.x_out == nullptr) return;
+    ss = block_sum2(s1, 0.0f, scratch[2]);
+    const float f = 1.0f / sqrtf(ss.x / (float)width + a.next_eps);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        const int i = (threadIdx.x + r * blockDim.x) * VEC;
+        if (i < width) {
+            float w[VEC];
+            RowVec<float, VEC>::load(a.next_w + i, w);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) w[j] = u[r][j] * f * w[j];
+            row_store<TO, VEC>((TO*)a.x_out + base + i, w);
+        }
+    }
+}
+
+extern "C" int mf_norm_terms(const NormTermsArgs* args, int n_rows, int out_dtype, cudaStream_t stream) {
+    const NormTermsArgs a = *args;
+    if (n_rows <= 0) return 0;
+    const bool pair = a.t2.y != nullptr || a.t2.n_part > 0;
+    if (a.width < 1 || a.h == nullptr || a.t1.scale == nullptr || (a.t1.y == nullptr && a.t1.n_part <= 0)) return MF_ERR_ARGUMENT;
+    if ((a.t1.n_part > 0 && a.t1.part == nullptr) || (a.t2.n_part > 0 && a.t2.part == nullptr)) return MF_ERR_ARGUMENT;
+    if ((pair && a.t2.scale == nullptr) || (a.x_out != nullptr && a.next_w == nullptr)) return MF_ERR_ARGUMENT;
+    const uintptr_t ptrs = (uintptr_t)a.h | (uintptr_t)a.t1.y | (uintptr_t)a.t1.part | (uintptr_t)a.t1.scale |
+                           (uintptr_t)a.t2.y | (uintptr_t)a.t2.part | (uintptr_t)a.t2.scale | (uintptr_t)a.out_w |
+                           (uintptr_t)a.next_w | (uintptr_t)a.x_out;
+    const bool vec = (a.width & 3) == 0 && (ptrs & 15) == 0;
+    const int per = vec ? 4 : 1;
+    if (a.width > 4 * 1024 * per) return MF_ERR_UNSUPPORTED;
+    // (a function of the width only: a row's sums never depend on the batch)
+    int threads = 32;
+    while (threads < 1024 && threads * 2 * per < a.width) threads <<= 1;
+#define MF_NT2(T, V, P) mf_launch(norm_terms_kernel<T, V, P>, dim3(n_rows), dim3(threads), 0, stream, a)
+#define MF_NT(T, V) do { if (pair) MF_NT2(T, V, true); else MF_NT2(T, V, false); } while (0)
+    if (out_dtype == MF_DTYPE_F32) { if (vec) MF_NT(float, 4); else MF_NT(float, 1); }
+    else if (out_dtype == MF_DTYPE_BF16) { if (vec) MF_NT(__nv_bfloat16, 4); else MF_NT(__nv_bfloat16, 1); }
+    else return MF_ERR_UNSUPPORTED;
+#undef MF_NT
+#undef MF_NT2
     return MF_LAUNCH_CHECK();
 }

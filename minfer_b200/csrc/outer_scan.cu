@@ -9,7 +9,10 @@
 //                 n_t likewise with k_t alone;  out = S_t^T q_t,  den = max(|n_t . q_t|, e^(-m_t)) + 1e-6
 //                 (the division is the next kernel's, which norms each head anyway).  n is kept as
 //                 one more column of S, whose value is always 1.
+//   gla_scan      a decay per key channel, the current token's own pair included in what it reads:
+//                 S_t = diag(w_t) S_(t-1) + k_t v_t^T;  o_t = S_t^T q_t
 //   wkv_decay     w = exp(-exp(w0 + W2 tanh(t1))) per token and channel, W2 through a small rank
+//   sigmoid_decay w = sigmoid(w0 + W2 t1)^(1 / tau), likewise
 //
 // The scan: a block owns (row, head, a tile of columns).  Four warps walk the tokens: LD neighbouring
 // lanes share a pair of columns and hold its state elements d = 4 (l + LD i) .. + 3 in registers, so
@@ -32,16 +35,22 @@
 #define OS_STAGES 4
 #define OS_MAX_D 256
 
+// the recurrences; which of them have a decay per key channel, a bonus, gates with a running maximum
+enum OuterMode { OS_WKV = 0, OS_MLSTM = 1, OS_GLA = 2 };
+template <int MODE> struct OuterTraits {
+    static constexpr bool DECAYS = MODE != OS_MLSTM, BONUS = MODE == OS_WKV, GATES = MODE == OS_MLSTM;
+};
+
 struct OuterScanArgs {
     const float* r;          // read vectors (r or q): r[t * r_width + r_off + head * D + d]
     const float* k;
     const float* v;          // v[t * v_width + v_off + head * Dv + j]
-    const float* w;          // wkv: decays w[t * w_width + w_off + head * D + d]
+    const float* w;          // wkv, gla: decays w[t * w_width + w_off + head * D + d]
     const float* u;          // wkv: bonus [heads][D]
     const float* gates;      // mlstm: raw gates, gates[t * gate_width + i_off + head], .. f_off ..
     const float* i_bias;     // [heads]
     const float* f_bias;     // [heads]
-    float* state;            // [slots][heads][columns][D], columns Dv (wkv) or Dv + 1 (mlstm)
+    float* state;            // [slots][heads][columns][D], columns Dv or Dv + 1 (mlstm)
     float* maxima;           // mlstm: [slots][heads][Dv + 1]
     const int* cu_seqlens;
     const int* slots;
@@ -50,7 +59,7 @@ struct OuterScanArgs {
     long long r_width, k_width, v_width, w_width, gate_width;
     int r_off, k_off, v_off, w_off, i_off, f_off;
     int n_rows, heads, D, Dv;
-    float cap, r_scale;      // mlstm: cap of the gates; factor on q
+    float cap, r_scale;      // mlstm: cap of the gates; mlstm, gla: factor on q
 };
 
 __device__ __forceinline__ void os_cp4(float* dst, const float* src) {
@@ -92,7 +101,7 @@ __device__ __forceinline__ void os_bar_arrive(int id) {
 #define OS_EMPTY(stage) (1 + OS_STAGES + (stage))
 
 // One token on this thread's two columns: acc += (state read with r), state updated.
-template <int ND4, bool WKV>
+template <int ND4, int MODE>
 __device__ __forceinline__ void os_token(float4 (&S0)[ND4], float4 (&S1)[ND4], const float4* r4,
                                          const float4* k4, const float4* w4, float keep, float v0,
                                          float v1, int step, float& acc0, float& acc1) {
@@ -100,7 +109,17 @@ __device__ __forceinline__ void os_token(float4 (&S0)[ND4], float4 (&S1)[ND4], c
 #pragma unroll
     for (int i = 0; i < ND4; ++i) {
         const float4 rr = r4[i * step], kk = k4[i * step];
-        if (WKV) {
+        if (MODE == OS_GLA) {
+            const float4 ww = w4[i * step];
+            S0[i].x = fmaf(ww.x, S0[i].x, kk.x * v0); S1[i].x = fmaf(ww.x, S1[i].x, kk.x * v1);
+            S0[i].y = fmaf(ww.y, S0[i].y, kk.y * v0); S1[i].y = fmaf(ww.y, S1[i].y, kk.y * v1);
+            S0[i].z = fmaf(ww.z, S0[i].z, kk.z * v0); S1[i].z = fmaf(ww.z, S1[i].z, kk.z * v1);
+            S0[i].w = fmaf(ww.w, S0[i].w, kk.w * v0); S1[i].w = fmaf(ww.w, S1[i].w, kk.w * v1);
+            a0 = fmaf(rr.x, S0[i].x, a0); b0 = fmaf(rr.y, S0[i].y, b0);
+            a0 = fmaf(rr.z, S0[i].z, a0); b0 = fmaf(rr.w, S0[i].w, b0);
+            a1 = fmaf(rr.x, S1[i].x, a1); b1 = fmaf(rr.y, S1[i].y, b1);
+            a1 = fmaf(rr.z, S1[i].z, a1); b1 = fmaf(rr.w, S1[i].w, b1);
+        } else if (MODE == OS_WKV) {
             const float4 ww = w4[i * step];
             a0 = fmaf(rr.x, S0[i].x, a0); b0 = fmaf(rr.y, S0[i].y, b0);
             a0 = fmaf(rr.z, S0[i].z, a0); b0 = fmaf(rr.w, S0[i].w, b0);
@@ -129,17 +148,18 @@ __device__ __forceinline__ float os_soft_cap(float z, float cap) { return cap * 
 
 // LD: lanes that share a pair of columns; ND4: float4 groups of a column a lane holds (D <= 4 LD ND4);
 // tc: tokens of a chunk
-template <int LD, int ND4, bool WKV>
+template <int LD, int ND4, int MODE>
 __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(OuterScanArgs a, int tc) {
     pdl_launch_dependents();
     constexpr int DP = 4 * LD * ND4;                   // padded key size
     constexpr int TV = 2 * (OS_THREADS / LD);          // columns of a block
-    constexpr int NVEC = WKV ? 3 : 2;                  // vectors staged per token: r, k (and decays)
+    constexpr bool DECAYS = OuterTraits<MODE>::DECAYS, BONUS = OuterTraits<MODE>::BONUS, GATES = OuterTraits<MODE>::GATES;
+    constexpr int NVEC = DECAYS ? 3 : 2;               // vectors staged per token: r, k (and decays)
     extern __shared__ __align__(16) float os_smem[];
     // a stage: r k (w) | v | factors: wkv r . (u k), mlstm (decay, input) pairs and e^(-m)
     const int stage_floats = tc * (NVEC * DP + TV) + 4 * ((3 * tc + 3) / 4);
     const int D = a.D, Dv = a.Dv;
-    const int cols = WKV ? Dv : Dv + 1;
+    const int cols = GATES ? Dv + 1 : Dv;
     const int tiles = (cols + TV - 1) / TV;
     const int h = blockIdx.x / tiles, tile = blockIdx.x - h * tiles;
     const int b = blockIdx.y;
@@ -167,13 +187,13 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
             }
         }
         float ib = 0.f, fb = 0.f;
-        if (!WKV) { ib = a.i_bias[h]; fb = a.f_bias[h]; }
+        if (GATES) { ib = a.i_bias[h]; fb = a.f_bias[h]; }
         pdl_wait();
         float m_run = 0.f;
-        if (!WKV) m_run = a.maxima[((size_t)slot * a.heads + h) * cols + j0];
+        if (GATES) m_run = a.maxima[((size_t)slot * a.heads + h) * cols + j0];
         float raw_i[3] = {0.f, 0.f, 0.f}, raw_f[3] = {0.f, 0.f, 0.f};   // raw gates: this chunk's, the next two's
         float bonus[DP / 32];                          // (wkv) this lane's share of the head's bonus
-        if (WKV) {
+        if (BONUS) {
 #pragma unroll
             for (int e = 0; e < DP / 32; ++e) bonus[e] = lane + 32 * e < D ? a.u[h * D + lane + 32 * e] : 0.f;
         }
@@ -187,26 +207,26 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
             const size_t t = (size_t)(t0 + c0);
             const float* rg = a.r + t * a.r_width + a.r_off + h * D;
             const float* kg = a.k + t * a.k_width + a.k_off + h * D;
-            const float* wg = WKV ? a.w + t * a.w_width + a.w_off + h * D : nullptr;
+            const float* wg = DECAYS ? a.w + t * a.w_width + a.w_off + h * D : nullptr;
             const float* vg = a.v + t * a.v_width + a.v_off + (size_t)h * Dv + j0;
             r_s += fw * DP; k_s += fw * DP; w_s += fw * DP;
-            rg += fw * a.r_width; kg += fw * a.k_width; if (WKV) wg += fw * a.w_width;
+            rg += fw * a.r_width; kg += fw * a.k_width; if (DECAYS) wg += fw * a.w_width;
             for (int tt = fw; tt < nc; tt += OS_FEED) {
                 if (vec) {
                     for (int d = 4 * lane; d < D; d += 128) {
                         os_cp16(r_s + d, rg + d);
                         os_cp16(k_s + d, kg + d);
-                        if (WKV) os_cp16(w_s + d, wg + d);
+                        if (DECAYS) os_cp16(w_s + d, wg + d);
                     }
                 } else {
                     for (int d = lane; d < D; d += 32) {
                         os_cp4(r_s + d, rg + d);
                         os_cp4(k_s + d, kg + d);
-                        if (WKV) os_cp4(w_s + d, wg + d);
+                        if (DECAYS) os_cp4(w_s + d, wg + d);
                     }
                 }
                 r_s += OS_FEED * DP; k_s += OS_FEED * DP; w_s += OS_FEED * DP;
-                rg += OS_FEED * a.r_width; kg += OS_FEED * a.k_width; if (WKV) wg += OS_FEED * a.w_width;
+                rg += OS_FEED * a.r_width; kg += OS_FEED * a.k_width; if (DECAYS) wg += OS_FEED * a.w_width;
             }
             if (vec_v && (v_cols & 3) == 0) {
                 const int per = v_cols >> 2;
@@ -220,7 +240,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
                     os_cp4(v_s + tt * TV + cc, vg + (size_t)tt * a.v_width + cc);
                 }
             }
-            if (!WKV && fw == 0) {
+            if (GATES && fw == 0) {
                 if (j0 + n_cols == cols)               // the normalizer's column
                     for (int tt = lane; tt < nc; tt += 32) v_s[tt * TV + n_cols - 1] = 1.0f;
                 raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1];
@@ -235,7 +255,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
         // two chunks ahead; a chunk that does not exist is an empty group of copies
         for (int ahead = 0; ahead < 2; ++ahead) {
             if (ahead < n_chunks) fetch(ahead);
-            else if (!WKV) { raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1]; raw_i[1] = raw_i[2]; raw_f[1] = raw_f[2]; }
+            else if (GATES) { raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1]; raw_i[1] = raw_i[2]; raw_f[1] = raw_f[2]; }
             asm volatile("cp.async.commit_group;" ::: "memory");
         }
         for (int chunk = 0; chunk < n_chunks; ++chunk) {
@@ -243,7 +263,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
             if (chunk + 2 < n_chunks) {
                 if (chunk + 2 >= OS_STAGES) os_bar_sync(OS_EMPTY((chunk + 2) % OS_STAGES));
                 fetch(chunk + 2);
-            } else if (!WKV) {
+            } else if (GATES) {
                 raw_i[0] = raw_i[1]; raw_f[0] = raw_f[1];
                 raw_i[1] = raw_i[2]; raw_f[1] = raw_f[2];
             }
@@ -253,7 +273,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
             float* r_s = os_smem + (chunk % OS_STAGES) * stage_floats;
             float* k_s = r_s + tc * DP;
             float* f_s = r_s + tc * (NVEC * DP + TV);
-            if (WKV) {
+            if (BONUS) {
                 // r . (u k), of the tokens this warp copied: what the current token's own value is
                 // multiplied by
                 constexpr int OWN = OS_TC / OS_FEED;
@@ -281,7 +301,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
                     for (int i = 0; i < OWN; ++i)
                         if (fw + OS_FEED * i < nc) f_s[fw + OS_FEED * i] = s[i];
                 }
-            } else if (fw == 0) {
+            } else if (GATES && fw == 0) {
                 // a token a lane; the maxima by a scan in which a stretch of tokens is the pair
                 // (sum of f, largest i + the f's after it)
                 const bool mine = lane < nc;
@@ -308,7 +328,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
             }
             os_bar_arrive(OS_FULL(chunk % OS_STAGES));
         }
-        if (!WKV && fw == 0)
+        if (GATES && fw == 0)
             for (int i = lane; i < n_cols; i += 32) a.maxima[((size_t)slot * a.heads + h) * cols + j0 + i] = m_run;
         return;
     }
@@ -345,7 +365,7 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
     // number `x` is the sum of token t (of the chunk, whose first token's output row is o) and column cc
     auto emit = [&](float x, float* o, const float* v_s, const float* f_s, int t, int cc, int token) {
         if (cc >= n_cols) return;
-        if (WKV) o[t * out_row + cc] = fmaf(f_s[t], v_s[t * TV + cc], x);
+        if (BONUS) o[t * out_row + cc] = fmaf(f_s[t], v_s[t * TV + cc], x);
         else if (j0 + cc < Dv) o[t * out_row + cc] = x * a.r_scale;
         else a.den[(size_t)(token + t) * a.heads + h] = fmaxf(fabsf(x * a.r_scale), f_s[2 * tc + t]) + 1e-6f;
     };
@@ -369,11 +389,11 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
                 const int t = tt + u;
                 float2 vv = *reinterpret_cast<const float2*>(v_s + t * TV + 2 * c);
                 float keep = 0.f;
-                if (!WKV) {
+                if (GATES) {
                     const float2 f = *reinterpret_cast<const float2*>(f_s + 2 * t);
                     keep = f.x; vv.x *= f.y; vv.y *= f.y;
                 }
-                os_token<ND4, WKV>(S0, S1, r4 + t * (DP / 4), k4 + t * (DP / 4), w4 + t * (DP / 4), keep, vv.x, vv.y, LD,
+                os_token<ND4, MODE>(S0, S1, r4 + t * (DP / 4), k4 + t * (DP / 4), w4 + t * (DP / 4), keep, vv.x, vv.y, LD,
                                    acc[2 * u], acc[2 * u + 1]);
             }
             os_reduce16<LD>(acc, l);
@@ -389,11 +409,11 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
         for (; tt < nc; ++tt) {
             float2 vv = *reinterpret_cast<const float2*>(v_s + tt * TV + 2 * c);
             float keep = 0.f, a0, a1;
-            if (!WKV) {
+            if (GATES) {
                 const float2 f = *reinterpret_cast<const float2*>(f_s + 2 * tt);
                 keep = f.x; vv.x *= f.y; vv.y *= f.y;
             }
-            os_token<ND4, WKV>(S0, S1, r4 + tt * (DP / 4), k4 + tt * (DP / 4), w4 + tt * (DP / 4), keep, vv.x, vv.y, LD, a0, a1);
+            os_token<ND4, MODE>(S0, S1, r4 + tt * (DP / 4), k4 + tt * (DP / 4), w4 + tt * (DP / 4), keep, vv.x, vv.y, LD, a0, a1);
 #pragma unroll
             for (int o2 = LD / 2; o2 > 0; o2 >>= 1) {
                 a0 += __shfl_xor_sync(0xffffffffu, a0, o2);
@@ -424,9 +444,9 @@ __global__ void __launch_bounds__(OS_THREADS + 32 * OS_FEED) outer_scan_kernel(O
     }
 }
 
-template <int LD, int ND4, bool WKV>
+template <int LD, int ND4, int MODE>
 static int os_launch(const OuterScanArgs& a, int max_tokens, cudaStream_t stream) {
-    constexpr int DP = 4 * LD * ND4, TV = 2 * (OS_THREADS / LD), NVEC = WKV ? 3 : 2;
+    constexpr int DP = 4 * LD * ND4, TV = 2 * (OS_THREADS / LD), NVEC = OuterTraits<MODE>::DECAYS ? 3 : 2;
     // (short rows take shorter chunks, so that more blocks fit an SM: single tokens most of all)
     const int tc = max_tokens < 1 ? OS_TC : max_tokens < OS_TC ? max_tokens : OS_TC;
     auto bytes = [&](int t) { return (size_t)OS_STAGES * (t * (NVEC * DP + TV) + 4 * ((3 * t + 3) / 4)) * sizeof(float); };
@@ -434,55 +454,61 @@ static int os_launch(const OuterScanArgs& a, int max_tokens, cudaStream_t stream
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return MF_ERR_UNSUPPORTED;
     if (!configured[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(outer_scan_kernel<LD, ND4, WKV>,
+        cudaError_t e = cudaFuncSetAttribute(outer_scan_kernel<LD, ND4, MODE>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes(OS_TC));
         if (e != cudaSuccess) return (int)e;
         configured[dev] = true;
     }
-    const int cols = WKV ? a.Dv : a.Dv + 1;
+    const int cols = OuterTraits<MODE>::GATES ? a.Dv + 1 : a.Dv;
     const int tiles = (cols + TV - 1) / TV;
-    mf_launch(outer_scan_kernel<LD, ND4, WKV>, dim3(a.heads * tiles, a.n_rows), dim3(OS_THREADS + 32 * OS_FEED), bytes(tc),
+    mf_launch(outer_scan_kernel<LD, ND4, MODE>, dim3(a.heads * tiles, a.n_rows), dim3(OS_THREADS + 32 * OS_FEED), bytes(tc),
               stream, a, tc);
     return MF_LAUNCH_CHECK();
 }
 
-template <bool WKV>
+template <int MODE>
 static int os_choose(const OuterScanArgs& a, int max_tokens, cudaStream_t stream) {
     if (a.n_rows <= 0) return 0;
     if (a.D < 1 || a.D > OS_MAX_D || a.Dv < 1 || a.heads < 1 || a.n_rows > 65535) return MF_ERR_UNSUPPORTED;
     if (((uintptr_t)a.state & 15) != 0) return MF_ERR_UNSUPPORTED;
-    if (a.D <= 32) return os_launch<8, 1, WKV>(a, max_tokens, stream);
-    if (a.D <= 64) return os_launch<16, 1, WKV>(a, max_tokens, stream);
-    if (a.D <= 128) return os_launch<16, 2, WKV>(a, max_tokens, stream);
-    return os_launch<32, 2, WKV>(a, max_tokens, stream);
+    if (a.D <= 32) return os_launch<8, 1, MODE>(a, max_tokens, stream);
+    if (a.D <= 64) return os_launch<16, 1, MODE>(a, max_tokens, stream);
+    if (a.D <= 128) return os_launch<16, 2, MODE>(a, max_tokens, stream);
+    return os_launch<32, 2, MODE>(a, max_tokens, stream);
 }
 
 // max_tokens: the most tokens a row brings (0: not known; it only sizes the chunks)
 extern "C" int mf_wkv_scan(const OuterScanArgs* args, int max_tokens, cudaStream_t stream) {
-    return os_choose<true>(*args, max_tokens, stream);
+    return os_choose<OS_WKV>(*args, max_tokens, stream);
 }
 extern "C" int mf_mlstm_scan(const OuterScanArgs* args, int max_tokens, cudaStream_t stream) {
     if (!(args->cap > 0.0f)) return MF_ERR_ARGUMENT;
-    return os_choose<false>(*args, max_tokens, stream);
+    return os_choose<OS_MLSTM>(*args, max_tokens, stream);
+}
+extern "C" int mf_gla_scan(const OuterScanArgs* args, int max_tokens, cudaStream_t stream) {
+    return os_choose<OS_GLA>(*args, max_tokens, stream);
 }
 
 // ------------------------------------------------------------------------------------------
-// out[t][c] = exp(-exp(w0[c] + sum_r w2t[r][c] tanh(t1[t][r]))): a thread per channel, WD_T tokens a
-// block, whose tanh(t1) lie in shared memory.
+// out[t][c] = exp(-exp(w0[c] + sum_r w2t[r][c] tanh(t1[t][r]))) or, SIGMOID, with z = w0[c] + sum_r
+// w2t[r][c] t1[t][r], sigmoid(z)^inv_tau = exp(inv_tau log sigmoid(z)): a thread per channel, WD_T
+// tokens a block, whose tanh(t1) (t1) lie in shared memory.
 // ------------------------------------------------------------------------------------------
 #define WD_T 16
 
-template <int NT>
+template <int NT, bool SIGMOID>
 __global__ void __launch_bounds__(128)
-wkv_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* __restrict__ w2t,
-                 const float* __restrict__ w0, float* __restrict__ out, int n_tokens, int rank, int channels) {
+low_rank_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* __restrict__ w2t,
+                 const float* __restrict__ w0, float* __restrict__ out, int n_tokens, int rank, int channels,
+                      float inv_tau) {
     pdl_prologue();
     extern __shared__ __align__(16) float wd_s[];      // [NT][rank, padded to a multiple of 4]
     const int first = blockIdx.y * NT, nt = min(NT, n_tokens - first);
     const int pitch = (rank + 3) & ~3;
     for (int i = threadIdx.x; i < NT * rank; i += blockDim.x) {
         const int t = i / rank, r = i - t * rank;
-        wd_s[t * pitch + r] = t < nt ? tanhf(t1[(size_t)(first + t) * t1_width + r]) : 0.f;
+        const float x = t < nt ? t1[(size_t)(first + t) * t1_width + r] : 0.f;
+        wd_s[t * pitch + r] = SIGMOID ? x : tanhf(x);
     }
     __syncthreads();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -518,22 +544,34 @@ wkv_decay_kernel(const float* __restrict__ t1, long long t1_width, const float* 
     }
 #pragma unroll
     for (int t = 0; t < NT; ++t)
-        if (t < nt) out[(size_t)(first + t) * channels + c] = expf(-expf(acc[t]));
+        if (t < nt)
+            out[(size_t)(first + t) * channels + c] =
+                SIGMOID ? expf(inv_tau * (fminf(acc[t], 0.f) - log1pf(expf(-fabsf(acc[t]))))) : expf(-expf(acc[t]));
 }
 
-extern "C" int mf_wkv_decay(const float* t1, long long t1_width, const float* w2t, const float* w0,
-                            float* out, int n_tokens, int rank, int channels, cudaStream_t stream) {
+template <bool SIGMOID>
+static int low_rank_decay(const float* t1, long long t1_width, const float* w2t, const float* w0, float* out,
+                          int n_tokens, int rank, int channels, float inv_tau, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank < 1 || channels < 1 || (size_t)(rank + 3) * WD_T * sizeof(float) > 48 * 1024) return MF_ERR_UNSUPPORTED;
     const int cb = (channels + 127) / 128;
     if (n_tokens <= 64) {
         if ((n_tokens + 1) / 2 > 65535) return MF_ERR_UNSUPPORTED;
-        mf_launch(wkv_decay_kernel<2>, dim3(cb, (n_tokens + 1) / 2), dim3(128), (size_t)((rank + 3) & ~3) * 2 * sizeof(float),
-                  stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels);
+        mf_launch(low_rank_decay_kernel<2, SIGMOID>, dim3(cb, (n_tokens + 1) / 2), dim3(128), (size_t)((rank + 3) & ~3) * 2 * sizeof(float),
+                  stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels, inv_tau);
     } else {
         if ((n_tokens + WD_T - 1) / WD_T > 65535) return MF_ERR_UNSUPPORTED;
-        mf_launch(wkv_decay_kernel<WD_T>, dim3(cb, (n_tokens + WD_T - 1) / WD_T), dim3(128),
-                  (size_t)((rank + 3) & ~3) * WD_T * sizeof(float), stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels);
+        mf_launch(low_rank_decay_kernel<WD_T, SIGMOID>, dim3(cb, (n_tokens + WD_T - 1) / WD_T), dim3(128),
+                  (size_t)((rank + 3) & ~3) * WD_T * sizeof(float), stream, t1, t1_width, w2t, w0, out, n_tokens, rank, channels, inv_tau);
     }
     return MF_LAUNCH_CHECK();
+}
+
+extern "C" int mf_wkv_decay(const float* t1, long long t1_width, const float* w2t, const float* w0,
+                            float* out, int n_tokens, int rank, int channels, cudaStream_t stream) {
+    return low_rank_decay<false>(t1, t1_width, w2t, w0, out, n_tokens, rank, channels, 1.0f, stream);
+}
+extern "C" int mf_sigmoid_decay(const float* t1, long long t1_width, const float* w2t, const float* w0, float* out,
+                                int n_tokens, int rank, int channels, float inv_tau, cudaStream_t stream) {
+    return low_rank_decay<true>(t1, t1_width, w2t, w0, out, n_tokens, rank, channels, inv_tau, stream);
 }

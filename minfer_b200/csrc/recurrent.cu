@@ -6,7 +6,8 @@
 // Tokens are packed row after row (row b: tokens cu_seqlens[b] .. cu_seqlens[b + 1]); a row goes
 // on from what its slot's state holds, so a step may bring any number of tokens per row.
 //
-//   conv_silu         u[t][c] = silu(bias[c] + sum_j taps[c][j] * in[t - (T - 1 - j)][c]) over the
+//   conv_silu         u[t][c] = act(bias[c] + sum_j taps[c][j] * in[t - (T - 1 - j)][c]), act silu or
+//                     (`plain`) nothing, over the
 //                     channels c of x | B | C; inputs before the row's first token come from the
 //                     slot's state (the last T - 1 inputs, oldest first; zeros for a new sequence)
 //                     (a thread per token and channel for single tokens; for longer rows a
@@ -38,7 +39,7 @@ conv_silu_kernel(const float* __restrict__ proj, long long in_width, int x_off, 
                  int taps, const float* __restrict__ w, const float* __restrict__ bias,
                  float* __restrict__ state, const int* __restrict__ token_row,
                  const int* __restrict__ cu_seqlens, const int* __restrict__ slots,
-                 float* __restrict__ out, long long total, int single) {
+                 float* __restrict__ out, long long total, int single, int plain) {
     pdl_launch_dependents();
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -63,7 +64,7 @@ conv_silu_kernel(const float* __restrict__ proj, long long in_width, int x_off, 
             if (j == taps - 1) in_cur = v;
         }
     }
-    out[idx] = rc_silu(acc);
+    out[idx] = plain ? acc : rc_silu(acc);
     if (single && taps > 1) {
         // this thread alone owns the (slot, channel): shift and append
         float old[RC_MAX_TAPS];
@@ -85,7 +86,7 @@ conv_silu_run_kernel(const float* __restrict__ proj, long long in_width, int x_o
                      int taps, const float* __restrict__ w, const float* __restrict__ bias,
                      const float* __restrict__ state, const int* __restrict__ token_row,
                      const int* __restrict__ cu_seqlens, const int* __restrict__ slots,
-                     float* __restrict__ out, int n_tokens) {
+                     float* __restrict__ out, int n_tokens, int plain) {
     pdl_launch_dependents();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= channels) return;
@@ -118,7 +119,7 @@ conv_silu_run_kernel(const float* __restrict__ proj, long long in_width, int x_o
         for (int j = 0; j < RC_MAX_TAPS; ++j)
             if (j < taps - 1) acc = fmaf(wt[j], hist[j], acc);
         acc = fmaf(wt[taps - 1], v, acc);
-        out[(size_t)t * channels + c] = rc_silu(acc);
+        out[(size_t)t * channels + c] = plain ? acc : rc_silu(acc);
 #pragma unroll
         for (int j = 0; j < RC_MAX_TAPS - 1; ++j)
             if (j < taps - 1) hist[j] = j + 1 < taps - 1 ? hist[j + 1] : v;
@@ -155,18 +156,18 @@ conv_state_kernel(const float* __restrict__ proj, long long in_width, int x_off,
 extern "C" int mf_conv_silu(const float* proj, long long in_width, int x_off, int channels, int taps,
                             const float* w, const float* bias, float* state, const int* token_row,
                             const int* cu_seqlens, const int* slots, float* out, int n_tokens,
-                            int n_rows, int single, cudaStream_t stream) {
+                            int n_rows, int single, int plain, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (taps < 1 || taps > RC_MAX_TAPS || channels < 1) return MF_ERR_UNSUPPORTED;
     const long long total = (long long)n_tokens * channels;
     if (single || n_tokens < RC_CONV_TB)
         mf_launch(conv_silu_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, proj,
                   in_width, x_off, channels, taps, w, bias, state, token_row, cu_seqlens, slots, out,
-                  total, single);
+                  total, single, plain);
     else
         mf_launch(conv_silu_run_kernel, dim3((channels + 255) / 256, (n_tokens + RC_CONV_TB - 1) / RC_CONV_TB),
                   dim3(256), 0, stream, proj, in_width, x_off, channels, taps, w, bias, (const float*)state,
-                  token_row, cu_seqlens, slots, out, n_tokens);
+                  token_row, cu_seqlens, slots, out, n_tokens, plain);
     if (!single && taps > 1) {
         const long long per_row = (long long)n_rows * channels;
         mf_launch(conv_state_kernel, dim3((unsigned)((per_row + 255) / 256)), dim3(256), 0, stream,

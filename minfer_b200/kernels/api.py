@@ -131,6 +131,7 @@ def _sig_ops(lib: ctypes.CDLL) -> None:
                                  [c_int, c_int, c_void_p])
     lib.mf_scaled_add.argtypes = ([c_void_p] + [c_void_p, c_void_p, c_int, c_void_p] * 2 +
                                   [c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p])
+    lib.mf_norm_terms.argtypes = [c_void_p, c_int, c_int, c_void_p]
 
 
 def _sig_gemm_simt(lib: ctypes.CDLL) -> None:
@@ -203,8 +204,8 @@ def _sig_gemm_tc(lib: ctypes.CDLL) -> None:
                                        c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float,
                                        c_float, c_void_p, c_void_p]
     lib.mf_gemm_tc_xielu.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong,
-                                     c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int,
-                                     c_int, c_float, c_void_p, c_void_p]
+                                     c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p,
+                                     c_int, c_int, c_float, c_void_p, c_void_p]
     lib.mf_gemm_tc_gated.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong,
                                      c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p]
     lib.mf_gemm_tc_prep_parts.argtypes = [c_int, c_int, c_int]
@@ -227,7 +228,7 @@ def _sig_attention_prefill_tc(lib: ctypes.CDLL) -> None:
 
 def _sig_recurrent(lib: ctypes.CDLL) -> None:
     lib.mf_conv_silu.argtypes = ([c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 7 +
-                                 [c_int, c_int, c_int, c_void_p])
+                                 [c_int, c_int, c_int, c_int, c_void_p])
     lib.mf_ssm_scan.argtypes = ([c_void_p, c_void_p, c_longlong, c_int, c_int] + [c_void_p] * 7 +
                                 [c_int] * 6 + [c_void_p])
     lib.mf_gated_group_norm.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p,
@@ -245,6 +246,9 @@ def _sig_retention(lib: ctypes.CDLL) -> None:
 def _sig_outer_scan(lib: ctypes.CDLL) -> None:
     lib.mf_wkv_scan.argtypes = [c_void_p, c_int, c_void_p]
     lib.mf_mlstm_scan.argtypes = [c_void_p, c_int, c_void_p]
+    lib.mf_gla_scan.argtypes = [c_void_p, c_int, c_void_p]
+    lib.mf_sigmoid_decay.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                     c_int, c_float, c_void_p]
     lib.mf_wkv_decay.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                  c_int, c_void_p]
 
@@ -610,10 +614,11 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
 
 
 def gemm_tc_xielu(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act_p: float, act_n: float,
-                  status: torch.Tensor, row_scale: Optional["RowScale"] = None) -> None:
-    """out = f(x @ w^T) on tcgen05, f the xIELU activation with its two coefficients
-    (act_p = softplus(a0), act_n = 1/2 + softplus(a1)) applied to the float32 sums in the
-    product's epilogue.  ``row_scale`` as in ``gemm_tc_fused``."""
+                  status: torch.Tensor, row_scale: Optional["RowScale"] = None, act_l: float = 0.5) -> None:
+    """out = f(x @ w^T) on tcgen05, f(z) = act_p z^2 + act_l z (z > 0), act_n (exp(z) - 1 - z) + act_l z
+    (z <= 0), applied to the float32 sums in the product's epilogue: the xIELU activation (act_p =
+    softplus(a0), act_n = 1/2 + softplus(a1), act_l = 1/2) or the square of relu (1, 0, 0).
+    ``row_scale`` as in ``gemm_tc_fused``."""
     m, k = x.shape
     n = w.shape[0]
     if w.shape[1] != k or out.shape != (m, n) or out.stride(1) != 1:
@@ -626,7 +631,7 @@ def gemm_tc_xielu(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act_p: fl
         raise KernelError("gemm: the sums of squares must be [parts, rows]")
     _check(_lib("gemm_tc").mf_gemm_tc_xielu(
         x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0),
-        dtype_code(out.dtype), m, n, k, float(act_p), float(act_n),
+        dtype_code(out.dtype), m, n, k, float(act_p), float(act_n), float(act_l),
         _f32(rs.ssq, "ssq") if rs is not None else None, rs.ssq.shape[0] if rs is not None else 0,
         rs.width if rs is not None else 0, rs.eps if rs is not None else 0.0,
         _i32(status, "status"), _stream()), "gemm_tc_xielu")
@@ -917,8 +922,9 @@ def attention_paged(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
 def conv_silu(proj: torch.Tensor, x_off: int, channels: int, weight: torch.Tensor,
               bias: Optional[torch.Tensor], state: torch.Tensor, token_row: torch.Tensor,
               cu_seqlens: torch.Tensor, slots: torch.Tensor, out: torch.Tensor, n_rows: int,
-              single: bool) -> None:
-    """out[t][c] = silu(bias[c] + sum_j weight[c][j] * in[t - (taps - 1 - j)][c]) over the columns
+              single: bool, activation: str = "silu") -> None:
+    """out[t][c] = act(bias[c] + sum_j weight[c][j] * in[t - (taps - 1 - j)][c]), act silu or
+    ("none") nothing, over the columns
     x_off .. x_off + channels of ``proj`` (float32 [tokens, width]); inputs before a row's first
     token come from ``state`` [slots, channels, taps - 1], which then takes the row's last ones."""
     n = proj.shape[0]
@@ -926,11 +932,13 @@ def conv_silu(proj: torch.Tensor, x_off: int, channels: int, weight: torch.Tenso
     if (weight.shape[0] != channels or out.shape != (n, channels) or state.shape[1:] != (channels, max(taps - 1, 0))
             or x_off + channels > proj.shape[1]):
         raise KernelError("conv_silu: shapes do not fit")
+    if activation not in ("silu", "none"):
+        raise KernelError(f"conv_silu: the activation is silu or none, got {activation!r}")
     _check(_lib("recurrent").mf_conv_silu(
         _f32(proj, "proj"), proj.shape[1], int(x_off), int(channels), int(taps), _f32(weight, "weight"),
         _f32(bias, "bias"), _f32(state, "state"), _i32(token_row, "token_row"),
         _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), _f32(out, "out"), n, int(n_rows),
-        1 if single else 0, _stream()), "conv_silu", 1 if single or taps < 2 else 2)
+        1 if single else 0, 1 if activation == "none" else 0, _stream()), "conv_silu", 1 if single or taps < 2 else 2)
 
 
 def ssm_scan(u: torch.Tensor, proj: torch.Tensor, dt_off: int, dt_bias: torch.Tensor,
@@ -1491,12 +1499,52 @@ def scaled_add(h: torch.Tensor, first, second=None, norm_weight: Optional[torch.
                                      _stream()), "scaled_add")
 
 
-UNARY_ACTIVATIONS = {"gelu": 0}
+class _ScaledTerm(ctypes.Structure):
+    _fields_ = [("y", c_void_p), ("part", c_void_p), ("n_part", c_int), ("scale", c_void_p)]
+
+
+class _NormTermsArgs(ctypes.Structure):
+    _fields_ = ([("h", c_void_p), ("t1", _ScaledTerm), ("t2", _ScaledTerm)] +
+                [(n, c_void_p) for n in ("out_w", "next_w", "x_out")] + [("width", c_int)] +
+                [(n, c_float) for n in ("mult", "eps", "out_eps", "next_eps")])
+
+
+def norm_terms(h: torch.Tensor, terms, eps: float, mult: float = 1.0, out_norm=None, next_norm=None,
+               x_out: Optional[torch.Tensor] = None) -> None:
+    """h[t] += N(mult * sum_k T_k[t] / rms(T_k[t]) * w_k) for one or two terms (y, partial, w): ``y`` float32
+    [rows, width] or None, the K splits ``partial`` [splits, rows, width] of a product or None, added in
+    split order, ``w`` float32 [width]; ``eps`` inside the root.  N is the norm ``out_norm`` (weight, eps),
+    or nothing.  With ``x_out`` (the type of the activations) and ``next_norm`` (weight, eps): x_out =
+    h / rms(h) * weight, the norm that reads the new h next."""
+    n, width = h.shape
+    if not 1 <= len(terms) <= 2:
+        raise KernelError("norm_terms: one or two terms")
+    a = _NormTermsArgs()
+    for slot, (y, partial, w) in zip((a.t1, a.t2), terms):
+        if ((y is None and partial is None) or (y is not None and y.shape != h.shape) or w.numel() != width
+                or (partial is not None and (partial.dim() != 3 or partial.shape[1:] != h.shape))):
+            raise KernelError("norm_terms: shapes do not fit")
+        slot.y, slot.part, slot.scale = _f32(y, "y"), _f32(partial, "partial"), _f32(w, "w")
+        slot.n_part = partial.shape[0] if partial is not None else 0
+    a.h, a.width, a.mult, a.eps = _f32(h, "h"), width, float(mult), float(eps)
+    if out_norm is not None:
+        a.out_w, a.out_eps = _f32(out_norm[0], "out_norm"), float(out_norm[1])
+    if x_out is not None:
+        if x_out.shape != h.shape or next_norm is None or next_norm[0].numel() != width:
+            raise KernelError("norm_terms: the next norm does not fit the stream")
+        a.next_w, a.next_eps = _f32(next_norm[0], "next_norm"), float(next_norm[1])
+        a.x_out = _ptr(x_out, "x_out")
+    _check(_lib("ops").mf_norm_terms(ctypes.addressof(a), n, dtype_code(x_out.dtype) if x_out is not None else F32,
+                                     _stream()), "norm_terms")
+
+
+UNARY_ACTIVATIONS = {"gelu": 0, "relu2": 1}
 GATED_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
 
 
 def unary_act(z: torch.Tensor, out: torch.Tensor, activation: str) -> None:
-    """out = act(z), z float32; "gelu" is the erf form 0.5 z (1 + erf(z / sqrt 2))."""
+    """out = act(z), z float32; "gelu" is the erf form 0.5 z (1 + erf(z / sqrt 2)), "relu2"
+    max(z, 0)^2."""
     if out.shape != z.shape:
         raise KernelError("unary_act: shapes do not fit")
     _check(_lib("ops").mf_unary_act(_f32(z, "z"), _ptr(out, "out"), dtype_code(out.dtype), z.numel(),
@@ -1710,6 +1758,43 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Ten
     a.n_rows, a.heads, a.D, a.Dv = int(n_rows), heads, d, dv
     a.r_scale = 1.0
     _check(_lib("outer_scan").mf_wkv_scan(ctypes.addressof(a), int(max_tokens), _stream()), "wkv_scan")
+
+
+def sigmoid_decay(t1: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, tau: float, out: torch.Tensor) -> None:
+    """out[t][c] = sigmoid(w0[c] + sum_r w2t[r][c] t1[t][r])^(1 / tau), all float32: ``t1`` [tokens, rank]
+    (rows may be strided), ``w2t`` [rank, channels]."""
+    n, rank = t1.shape
+    channels = w0.numel()
+    if w2t.shape != (rank, channels) or out.shape != (n, channels) or t1.stride(1) != 1:
+        raise KernelError("sigmoid_decay: shapes do not fit")
+    if not t1.is_cuda or t1.dtype != torch.float32 or not tau > 0.0:
+        raise KernelError("sigmoid_decay: t1 must be float32 on a CUDA device, tau positive")
+    _check(_lib("outer_scan").mf_sigmoid_decay(t1.data_ptr(), t1.stride(0), _f32(w2t, "w2t"), _f32(w0, "w0"),
+                                               _f32(out, "out"), n, rank, channels, 1.0 / float(tau),
+                                               _stream()), "sigmoid_decay")
+
+
+def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, q_scale: float,
+             state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
+             n_rows: int, max_tokens: int = 0) -> None:
+    """Gated linear attention per (row, head), tokens one after another, from the columns of the float32
+    rows ``proj`` (q and k heads of D, v heads of Dv): S <- diag(decay) S + k v^T, then out = q_scale S^T q.
+    ``decay`` float32 [tokens, heads * D], ``out`` [tokens, heads * Dv]; S float32 in ``state`` [slots,
+    heads, Dv, D].  ``max_tokens``: the most tokens a row brings (0: not known)."""
+    n = proj.shape[0]
+    _, heads, dv, d = state.shape
+    if (out.shape != (n, heads * dv) or decay.shape != (n, heads * d)
+            or max(max(q_off, k_off) + heads * d, v_off + heads * dv) > proj.shape[1]):
+        raise KernelError("gla_scan: shapes do not fit")
+    a = _OuterScanArgs()
+    a.r = a.k = a.v = _f32(proj, "proj")
+    a.r_width = a.k_width = a.v_width = proj.shape[1]
+    a.r_off, a.k_off, a.v_off = int(q_off), int(k_off), int(v_off)
+    a.w, a.w_width, a.state = _f32(decay, "decay"), heads * d, _f32(state, "state")
+    a.cu_seqlens, a.slots, a.out = _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), _f32(out, "out")
+    a.n_rows, a.heads, a.D, a.Dv = int(n_rows), heads, d, dv
+    a.r_scale = float(q_scale)
+    _check(_lib("outer_scan").mf_gla_scan(ctypes.addressof(a), int(max_tokens), _stream()), "gla_scan")
 
 
 def mlstm_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off: int, f_off: int,

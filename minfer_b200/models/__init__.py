@@ -2,6 +2,7 @@
 from ..config.bedarax import ARCHITECTURE as BEDARAX, BedaraxConfig
 from ..config.budanex import ARCHITECTURE as BUDANEX, BudanexConfig
 from ..config.furitar import ARCHITECTURE as FURITAR, FuritarConfig
+from ..config.pazatar import ARCHITECTURE as PAZATAR, PazatarConfig
 from ..config.pikavik import ARCHITECTURE as PIKAVIK, PikavikConfig
 from ..config.qwen2 import ARCHITECTURE as QWEN2, Qwen2Config
 from ..config.zanelorn import ARCHITECTURE as ZANELORN, ZanelornConfig
@@ -13,3 +14,4 @@ register_architecture(BUDANEX, BudanexConfig.from_dict, replace=True)
 register_architecture(BEDARAX, BedaraxConfig.from_dict, replace=True)
 register_architecture(ZANELORN, ZanelornConfig.from_dict, replace=True)
 register_architecture(PIKAVIK, PikavikConfig.from_dict, replace=True)
+register_architecture(PAZATAR, PazatarConfig.from_dict, replace=True)

@@ -3,8 +3,9 @@ from ..registry import register_part
 from .attention import Attention
 from .base import (Block, CacheRequest, CacheView, CallBinding, FeedForward, Mixer, Norm, Part,
                    PositionEncoding, StateRequest, StepContext)
-from .block import OutputNormBlock, ParallelBlock, PreNormBlock, TokenSide
+from .block import OutputNormBlock, ParallelBlock, PreNormBlock, SandwichNormBlock, TokenSide
 from .delta_rule import GatedDeltaRule
+from .gated_linear import GatedLinearAttention
 from .latent_attention import LatentAttention
 from .linear import Linear
 from .mamba2 import Mamba2
@@ -39,6 +40,7 @@ register_part("mixer", "selective_scan", SelectiveScan, replace=True)
 register_part("mixer", "parallel", ParallelMixer, replace=True)
 register_part("mixer", "wkv", Wkv, replace=True)
 register_part("mixer", "mlstm", MLstm, replace=True)
+register_part("mixer", "gated_linear_attention", GatedLinearAttention, replace=True)
 register_part("feed_forward", "gated_mlp", GatedMlp, replace=True)
 register_part("feed_forward", "dense_mlp", DenseMlp, replace=True)
 register_part("feed_forward", "routed_experts", RoutedExperts, replace=True)
@@ -52,4 +54,6 @@ register_part("block", "pre_norm", lambda layer, **options: PreNormBlock(layer, 
 register_part("block", "output_norm", lambda layer, **options: OutputNormBlock(layer, **options),
               replace=True)
 register_part("block", "parallel", lambda layer, **options: ParallelBlock(layer, **options),
+              replace=True)
+register_part("block", "sandwich_norm", lambda layer, **options: SandwichNormBlock(layer, **options),
               replace=True)

@@ -398,3 +398,92 @@ class ParallelBlock(Block):
         K.scaled_add(h, (y, partial, self.scales[0]), second, weight, eps, x_out)
         if x_out is not None:
             ctx.extras["prepared"] = Prepared(x_out, None, target)
+
+
+class SandwichNormBlock(Block):
+    """A block that norms before and after each sublayer:
+
+        h += norm1b(mixer(norm1(h)));   h += norm2b(ffn(norm2(h)))            (the second half optional)
+
+    ``output_norms``: the specs of norm1b and norm2b (RMS norms).  A sublayer writes a buffer of its own, or
+    leaves the K splits of its last product, or (``offers_terms``) the terms its output is the sum of; one
+    kernel then norms that, adds it into the stream and norms the stream for whoever reads it next."""
+
+    capturable = True      # launches kernels only; safe inside a CUDA graph capture
+    accepts_pending = True     # a projection another block left pending is added by the first norm
+
+    def __init__(self, layer: LayerSpec, output_norms: Sequence[Any]):
+        from ..registry import build_part
+        self.prefix = layer.prefix
+        self.width = int(layer.mixer_norm.params["size"])
+        self.mixer_norm = build_part("norm", layer.mixer_norm)
+        self.mixer = build_part("mixer", layer.mixer)
+        self.feed_forward_norm = self.feed_forward = self.feed_forward_out = None
+        self.mixer_out = build_part("norm", output_norms[0])
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = build_part("norm", layer.feed_forward_norm)
+            self.feed_forward = build_part("feed_forward", layer.feed_forward)
+            self.feed_forward_out = build_part("norm", output_norms[1])
+        for norm in (self.mixer_out, self.feed_forward_out):
+            if norm is not None and norm.foldable() is None:
+                raise ValueError("this block norms a sublayer's output itself: its norms must be RMS norms")
+
+    def parts(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_out, self.feed_forward_norm,
+                                 self.feed_forward, self.feed_forward_out) if p is not None)
+
+    tensor_specs = PreNormBlock.tensor_specs
+    load = PreNormBlock.load
+    export = PreNormBlock.export
+    _sublayer = ParallelBlock._sublayer
+
+    def libraries(self, dtype: torch.dtype) -> List[str]:
+        return ["ops"]
+
+    def entry_norm(self):
+        return self.mixer_norm if self.mixer_norm.foldable() is not None else None
+
+    @staticmethod
+    def _input(norm, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        """The norm's output: what the kernel before left for this very norm, else the norm as a kernel
+        (which also adds a pending projection output into ``h``)."""
+        prepared = ctx.extras.pop("prepared", None)
+        pending = ctx.extras.pop("pending", None)
+        if prepared is not None and prepared.norm is norm and prepared.scale is None:
+            return prepared.x
+        if pending is not None:
+            return norm.forward_settling(h, pending, ctx.act_dtype)
+        return norm.forward(h, ctx.act_dtype)
+
+    def _add(self, part, x: torch.Tensor, out_norm, next_norm, h: torch.Tensor, ctx: StepContext, *args) -> None:
+        """h += out_norm(part(x)); the input of ``next_norm`` (None: nobody's) is left prepared."""
+        from ..kernels import api as K
+        weight, eps, _ = out_norm.foldable()
+        if getattr(part, "offers_terms", False):
+            ctx.extras.pop("prepare_for", None)
+            ctx.input_scale = None
+            ctx.extras["takes_terms"] = True
+            part.forward_add(x, ctx, *args, None)
+            left = ctx.extras.pop("terms")
+            terms, term_eps, mult, outer = left.terms, left.eps, left.mult, (weight, eps)
+        else:
+            terms, term_eps, mult, outer = [self._sublayer(part, x, ctx, *args) + (weight,)], eps, 1.0, None
+        fold = next_norm.foldable() if next_norm is not None else None
+        if fold is None or fold[2] != self.width:
+            K.norm_terms(h, terms, term_eps, mult, outer)
+            return
+        x_out = torch.empty((h.shape[0], self.width), dtype=ctx.act_dtype, device=h.device)
+        K.norm_terms(h, terms, term_eps, mult, outer, (fold[0], fold[1]), x_out)
+        ctx.extras["prepared"] = Prepared(x_out, None, next_norm)
+
+    def mix(self, h: torch.Tensor, ctx: StepContext, binding: CallBinding) -> None:
+        x = self._input(self.mixer_norm, h, ctx)
+        # (the engine may drop rows of h before the feed-forward, which then norms what is left)
+        target = self.feed_forward_norm if ctx.extras.get("rows_stay", True) else None
+        self._add(self.mixer, x, self.mixer_out, target, h, ctx, binding)
+
+    def feed(self, h: torch.Tensor, ctx: StepContext) -> None:
+        if self.feed_forward is None:
+            return
+        x = self._input(self.feed_forward_norm, h, ctx)
+        self._add(self.feed_forward, x, self.feed_forward_out, ctx.extras.get("next_norm"), h, ctx)

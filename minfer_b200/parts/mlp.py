@@ -130,13 +130,15 @@ class DenseMlp(FeedForward):
     ``"gelu"``   the erf form 0.5 z (1 + erf(z / sqrt 2)), no learned numbers (and no tensor
                  ``act_name``), in float32 on the product's float32 sums.
 
+    ``"relu2"``  max(z, 0)^2, likewise.
+
     Tensor names are parameters (``up_name``, ``down_name``, ``act_name``, each behind the
     layer's prefix)."""
 
     capturable = True      # launches kernels only; safe inside a CUDA graph capture
     stores_fresh_output = True     # its last product goes through ``project_out``
-    ACTIVATIONS = ("xielu", "poly_norm", "gelu")
-    ACT_NUMBERS = {"xielu": 2, "poly_norm": 4, "gelu": 0}
+    ACTIVATIONS = ("xielu", "poly_norm", "gelu", "relu2")
+    ACT_NUMBERS = {"xielu": 2, "poly_norm": 4, "gelu": 0, "relu2": 0}
 
     def libraries(self, dtype: torch.dtype) -> List[str]:
         return ["ops", "gemm_tc"] if dtype == torch.bfloat16 else ["ops", "gemm_simt"]
@@ -174,12 +176,14 @@ class DenseMlp(FeedForward):
         self.act_params = (weights[f"{prefix}{self.act_name}"] if self.ACT_NUMBERS[self.activation]
                            else None)
         self.accepts_row_scale = self.up.takes_row_scale()
+        if self.activation == "relu2":
+            self._act_p, self._act_n, self._act_l = 1.0, 0.0, 0.0
         if self.activation != "xielu":
             return
         # the activation's two coefficients, once, for the product whose epilogue applies it
         a = self.act_params.detach().to("cpu", torch.float64)
         sp = torch.log1p(torch.exp(-a.abs())) + torch.clamp(a, min=0)
-        self._act_p, self._act_n = float(sp[0]), 0.5 + float(sp[1])
+        self._act_p, self._act_n, self._act_l = float(sp[0]), 0.5 + float(sp[1]), 0.5
 
     def export(self, prefix: str) -> Dict[str, torch.Tensor]:
         out = {f"{prefix}{self.up_name}": self.up.weight, f"{prefix}{self.down_name}": self.down.weight}
@@ -202,7 +206,10 @@ class DenseMlp(FeedForward):
                 and K.gemm_tc_supported(x, self.up.weight) and FUSE_ACTIVATION):
             # the activation rides on the up projection's epilogue
             K.gemm_tc_xielu(x, self.up.weight, act, self._act_p, self._act_n,
-                            gemm.status_word(x.device), row_scale=ctx.input_scale)
+                            gemm.status_word(x.device), row_scale=ctx.input_scale, act_l=self._act_l)
+        elif self.activation == "relu2":
+            z = self.up.forward(x, torch.float32, row_scale=ctx.input_scale)
+            K.unary_act(z, act, "relu2")
         else:
             z = self.up.forward(x, torch.float32, row_scale=ctx.input_scale)
             K.xielu(z, self.act_params, act)

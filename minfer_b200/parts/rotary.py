@@ -12,7 +12,10 @@ device, and its sine and cosine are float32.
 (turns over that context), pair i's frequency f_i becomes f_i / factor * ramp_i + f_i * (1 -
 ramp_i), ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), lo = max(floor(d(fast)), 0),
 hi = min(ceil(d(slow)), rotary_dim - 1), d(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta);
-cosine and sine are multiplied by 0.1 ln(factor) + 1 (``magnitude``).
+cosine and sine are multiplied by 0.1 ln(factor) + 1 (``magnitude``).  With ``low`` and ``high`` in the
+place of ``fast`` and ``slow`` (scaling by bands of wavelength l = 2 pi / f): f stays where
+l < original / high, becomes f / factor where l > original / low, and (1 - s) f / factor + s f with
+s = (original / l - low) / (high - low) between; no magnitude.
 """
 from __future__ import annotations
 
@@ -41,11 +44,13 @@ class Rotary(PositionEncoding):
         self.frequency_scale = float(frequency_scale)
         self.style = style
         self.scaling = None
+        self.by_bands = False
         if scaling is not None:
-            self.scaling = {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}
-            if not (self.scaling["factor"] > 0 and self.scaling["original"] > 0
-                    and self.scaling["fast"] > 0 and self.scaling["slow"] > 0):
-                raise ValueError("rotary scaling wants positive factor, original, fast and slow")
+            self.by_bands = "low" in scaling or "high" in scaling
+            keys = ("factor", "original") + (("low", "high") if self.by_bands else ("fast", "slow"))
+            self.scaling = {k: float(scaling[k]) for k in keys}
+            if not all(v > 0 for v in self.scaling.values()):
+                raise ValueError(f"rotary scaling wants positive {', '.join(keys)}")
         self._inv_freq: dict = {}
 
     def inverse_frequencies(self) -> torch.Tensor:
@@ -55,6 +60,11 @@ class Rotary(PositionEncoding):
         if self.scaling is None:
             return freq
         sc, dims = self.scaling, self.rotary_dim
+        if self.by_bands:
+            turns = sc["original"] * freq / (2.0 * math.pi)          # original / wavelength
+            s = (turns - sc["low"]) / (sc["high"] - sc["low"]) if sc["high"] != sc["low"] else torch.ones_like(turns)
+            blend = (1.0 - s) * freq / sc["factor"] + s * freq
+            return torch.where(turns > sc["high"], freq, torch.where(turns < sc["low"], freq / sc["factor"], blend))
 
         def dim_of(turns: float) -> float:
             return dims * math.log(sc["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
@@ -66,7 +76,7 @@ class Rotary(PositionEncoding):
 
     def magnitude(self) -> float:
         """The factor on every cosine and sine (1 without scaling)."""
-        return 1.0 if self.scaling is None else 0.1 * math.log(self.scaling["factor"]) + 1.0
+        return 1.0 if self.scaling is None or self.by_bands else 0.1 * math.log(self.scaling["factor"]) + 1.0
 
     def fused_rotary(self, device: torch.device) -> Optional[Tuple[torch.Tensor, int, int]]:
         if self.scaling is not None and self.magnitude() != 1.0:
