@@ -66,11 +66,10 @@ PAZ_C = {
                _ff(_att(2, 1, 64, 0.2, 64, 1e3, 64), 128)],
     "loop": {"start": 1, "stop": 2, "times": 2},
 }
-# many query heads on one key head, eight taps, a loop over all layers, keys of 128 with values of 96, one
-# state column and one decay channel
+# many query heads on one key head, eight taps, a loop over all layers, keys of 128 with values of 96
 PAZ_D = {
     "architecture": "Pazatar", "vocab": 173, "width": 128, "norm": {"eps": 1e-6},
-    "layers": [_ff(_par((20, 1, 24, 32, 0.3, 4.0, 8, 90, 2e3, 12, (5.0, 200, 2.0, 4.0)), (4, 1, 1, 3.0, 2)), 200),
+    "layers": [_ff(_par((20, 1, 24, 32, 0.3, 4.0, 8, 90, 2e3, 12, (5.0, 200, 2.0, 4.0)), (4, 24, 16, 11.0, 2)), 200),
                _ff(_par((2, 1, 128, 96, 0.1, 15.0, 5, 200, 6e4, 64, None), (1, 64, 128, 6.0, 40)), 72),
                _ff(_att(18, 1, 32, 0.25, 96, 700.0, 20), 152)],
     "loop": {"start": 0, "stop": 3, "times": 2},
