@@ -1605,6 +1605,258 @@ def workload_pikavik(args) -> int:
     return 0
 
 
+# ------------------------------------------------------------------------------------------
+# --workload pazatar: the Pazatar design beside the Qwen2 decoder at equal width and layers
+# ------------------------------------------------------------------------------------------
+# (name, width, attention heads, feed-forward width of Qwen2, heads of the gated linear attention): six
+# layers, attention and the parallel mixer in turn.  Heads of 128, four query heads a key head; chunks of
+# 8,192 positions (attention) and 1,024 (beside the recurrence, behind convolutions of 4 taps); gated linear
+# attention with keys of 128 and values of 256.  The feed-forward has two matrices instead of three and so
+# 3/2 of Qwen2's width
+PAZATAR_SIZES = [("w2048", 2048, 16, 5632, 8), ("w4096", 4096, 32, 11264, 16)]
+PAZATAR_LAYERS = 6
+
+
+def pazatar_config(width, heads, ff, gla_heads, vocab):
+    att = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    yarn = {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+    bands = {"factor": 8.0, "original": 8192, "low": 1.0, "high": 4.0}
+    mlp = {"kind": "dense", "ff": 3 * ff // 2}
+    first = {"type": "attention", "mlp": mlp,
+             "mixer": dict(att, mask={"size": 8192}, rot={"base": 500000.0, "dims": 128, "scaling": yarn})}
+    second = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": dict(att, softcap=50.0, conv=4, mask={"size": 1024},
+                     rot={"base": 500000.0, "dims": 64, "scaling": bands}),
+        "right": {"heads": gla_heads, "dim": 128, "vdim": 256, "tau": 16.0, "decay_rank": 16}}}
+    return {"architecture": "Pazatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": None,
+            "layers": [first, second] * (PAZATAR_LAYERS // 2)}
+
+
+def pazatar_prefill_flops(cfg, tokens):
+    """Matrix-product flops of one whole prompt (head on the last row only), the attention of the visible
+    keys, and the recurrence (per token and state element: decay, update and read-out)."""
+    w, n = cfg["width"], tokens
+    flops = 0.0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        a = m if layer["type"] == "attention" else m["left"]
+        h, kv, d, dv, c = a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["mask"]["size"]
+        own = 0 if layer["type"] == "attention" else kv * dv          # (the values are the keys)
+        per_token = 2 * w * (h * d + kv * d + own + h * dv)
+        pairs = sum(min(c, n - lo) * (min(c, n - lo) + 1) / 2 for lo in range(0, n, c))
+        flops += h * 2 * (d + dv) * pairs
+        if layer["type"] == "parallel":
+            r = m["right"]
+            nk, nv = r["heads"] * r["dim"], r["heads"] * r["vdim"]
+            per_token += 2 * w * (2 * nk + 3 * nv) + 2 * r["decay_rank"] * (w + nk) + 6 * nk * r["vdim"]
+        flops += (per_token + 4 * w * layer["mlp"]["ff"]) * n
+    return flops + 2 * w * cfg["vocab"]
+
+
+def pazatar_decode_bytes(model, cfg, batch, context_tokens):
+    """Bytes a decode step must read: the weights once (the embedding table as the head), the keys and
+    values of the chunk a position lies in, and the recurrent states (read and written)."""
+    total = model.parameter_bytes()
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        a = m if layer["type"] == "attention" else m["left"]
+        total += batch * (context_tokens % a["mask"]["size"]) * a["kv_heads"] * (a["dim"] + a["vdim"]) * 2
+        if layer["type"] == "parallel":
+            total += batch * 2 * m["right"]["heads"] * m["right"]["dim"] * m["right"]["vdim"] * 4
+    return total
+
+
+def pazatar_kernels(torch, K, pk, width, heads, ff, gla_heads, tokens=2048, batch=8):
+    """The design's own kernels alone (median of 20, L2 flushed before each): device time and the fraction
+    of the copy bandwidth (or of the product peak) their algorithmic bytes (flops) reach, each beside
+    the like kernel of another design at equal sizes."""
+    from minfer_b200.parts.base import CacheView, StepContext
+    from minfer_b200.parts.sink_attention import ScoreSpec, scored_attention
+    dev = "cuda:0"
+    bw = pk["hbm_gbs"] * 1e9
+    peak = pk["bf16_tflops"] * 1e12
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bf = torch.bfloat16
+    out = {}
+
+    def timed(name, fn, nbytes=None, flops=None):
+        ms = _median_ms(torch, fn, 20, flush)
+        out[name] = {"us": round(ms * 1e3, 1)}
+        if nbytes is not None:
+            out[name]["frac_of_copy"] = round(nbytes / (ms * 1e-3) / bw, 4)
+        if flops is not None:
+            out[name]["frac_of_product_peak"] = round(flops / (ms * 1e-3) / peak, 4)
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    def rnd(*shape):
+        return torch.randn(*shape, device=dev)
+
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    vec = torch.ones(width, device=dev)
+    nh, nk, hd = heads, heads // 4, 128
+    inv = torch.rand(64, dtype=torch.float64, device=dev)
+    for label, n, rows in (("prompt", tokens, 1), ("decode", batch, batch)):
+        per = n // rows
+        single = label == "decode"
+        cu, slots = i32([per * b for b in range(rows + 1)]), i32(list(range(rows)))
+        positions = i32([tokens + (t % per) if single else t for t in range(n)])
+        token_row = i32([t // per for t in range(n)])
+        ends = i32([tokens + 1 if single else tokens] * rows)
+        # ---- gated linear attention beside the like recurrences -----------------------------------------
+        H, D, Dv = gla_heads, 128, 256
+        nq, nv = H * D, H * Dv
+        proj = rnd(n, 2 * nq + 2 * nv + 16)
+        a2t, b2 = rnd(16, nq), rnd(nq)
+        decay, o = torch.empty(n, nq, device=dev), torch.empty(n, nv, device=dev)
+        timed(f"sigmoid_decay_{label}", lambda: K.sigmoid_decay(proj[:, 2 * nq + 2 * nv:], a2t, b2, 16.0, decay),
+              nbytes=n * (16 + nq) * 4 + 17 * nq * 4)
+        t1, w2t = rnd(n, 64), rnd(64, nq) * 0.1
+        timed(f"like:wkv_decay_{label}", lambda: K.wkv_decay(t1, w2t, b2, decay), nbytes=n * (64 + nq) * 4 + 65 * nq * 4)
+        K.sigmoid_decay(proj[:, 2 * nq + 2 * nv:], a2t, b2, 16.0, decay)
+        state = torch.zeros(rows, H, Dv, D, device=dev)
+        timed(f"gla_scan_{label}", lambda: K.gla_scan(proj, 0, nq, 2 * nq, decay, D ** -0.5, state, cu, slots, o, rows, per),
+              nbytes=n * (3 * nq + 2 * nv) * 4 + rows * 2 * nq * Dv * 4)
+        r, k, v, u = rnd(n, nq), rnd(n, nq) * 0.1, rnd(n, nv), rnd(H, D)
+        timed(f"like:wkv_scan_{label}", lambda: K.wkv_scan(r, k, v, decay, u, state, cu, slots, o, rows, per),
+              nbytes=n * (3 * nq + 2 * nv) * 4 + rows * 2 * nq * Dv * 4)
+        q2, k2, dec = rnd(n, H, D), rnd(n, H, D), torch.full((H,), 0.97, device=dev)
+        timed(f"like:retention_scan_{label}", lambda: K.retention_scan(q2, k2, proj, 2 * nq, dec, state, cu, slots, o, rows),
+              nbytes=n * (2 * nq + 2 * nv) * 4 + rows * 2 * nq * Dv * 4)
+        gated, nw = torch.empty(n, nv, dtype=bf, device=dev), torch.ones(nv, device=dev)
+        timed(f"unit_norm_gate_{label}", lambda: K.unit_norm_gate(o, proj, 2 * nq + nv, gated, H, 1e-6, "silu", weight=nw),
+              nbytes=n * nv * 10)
+        # ---- convolution, heads prepared -----------------------------------------------------------------
+        ch = (nh + 2 * nk) * hd
+        wide = rnd(n, ch + 2 * nq + 2 * nv + 16)
+        cw, cs, co = rnd(ch, 4), torch.zeros(rows, ch, 3, device=dev), torch.empty(n, ch, device=dev)
+        for name, act in (("conv", "none"), ("like:conv_silu", "silu")):
+            timed(f"{name}_{label}", lambda: K.conv_silu(wide, 0, ch, cw, None, cs, token_row, cu, slots, co, rows, single,
+                                                         activation=act), nbytes=n * ch * 8 + rows * ch * 24)
+        q, kk, vv = (torch.empty(n, x, hd, dtype=bf, device=dev) for x in (nh, nk, nk))
+        pages = tokens // 64 + 1
+        kc, vc = (rnd(rows * pages, nk, 64, hd).to(bf) for _ in range(2))
+        table = i32([[b * pages + p for p in range(pages)] for b in range(rows)])
+        nbytes = n * (ch * 4 + (nh + 2 * nk + (0 if single else 2 * nk)) * hd * 2)
+        qn, kn = torch.ones(nh * hd, device=dev), torch.ones(nk * hd, device=dev)
+        places = dict(q_off=0, n_heads=nh, q_width=hd, k_off=nh * hd, n_kv=nk, k_width=hd, v_width=hd, eps=1e-6, inv_freq=inv,
+                      rot_dims=hd, status=status)
+        step = (None, None) if single else (kk, vv)
+        timed(f"head_prepare_{label}", lambda: K.head_prepare(
+            co, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=(nh + nk) * hd, q_norm=qn[:hd],
+            k_norm=kn[:hd], rot_style=0, rot_magnitude=1.0, q_mul=1.0, k_mul=1.0, **places), nbytes=nbytes)
+        timed(f"qk_prepare_{label}", lambda: K.qk_prepare(
+            co, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=nh * hd, v_from_k=False, q_norm=qn,
+            k_norm=kn, rot_style=1, rot_magnitude=1.1, q_rot_off=0, k_rot_off=0, **places), nbytes=nbytes - n * nk * hd * 4)
+        timed(f"like:rope_kvstore_{label}", lambda: K.rope_kvstore(
+            co, positions, token_row, ends, inv, q, *step, kc, vc, table, pages, 0, nh, nk, hd, hd, 0, status), nbytes=nbytes)
+        # ---- the end of a sublayer -----------------------------------------------------------------------
+        h, y1, y2 = rnd(n, width), rnd(n, width), rnd(n, width)
+        xo = torch.empty(n, width, dtype=bf, device=dev)
+        timed(f"norm_terms_{label}", lambda: K.norm_terms(h, [(y1, None, vec)], 1e-6, 1.0, None, (vec, 1e-6), xo),
+              nbytes=n * width * 14)
+        timed(f"norm_terms_pair_{label}", lambda: K.norm_terms(h, [(y1, None, vec), (y2, None, vec)], 1e-6, 0.5, (vec, 1e-6),
+                                                               (vec, 1e-6), xo), nbytes=n * width * 18)
+        timed(f"like:norm_add_{label}", lambda: K.norm_add(h, y1, vec, 1e-6, 0.5, x_out=xo), nbytes=n * width * 14)
+        timed(f"like:scaled_add_{label}", lambda: K.scaled_add(h, (y1, None, vec), (y2, None, vec), vec, 1e-6, xo),
+              nbytes=n * width * 18)
+        # ---- relu squared in the up product's epilogue -----------------------------------------------------
+        x, wu = rnd(n, width).to(bf), rnd(3 * ff // 2, width).to(bf)
+        act = torch.empty(n, 3 * ff // 2, dtype=bf, device=dev)
+        cost = {"nbytes": wu.numel() * 2} if single else {"flops": 2.0 * n * wu.numel()}
+        timed(f"relu2_product_{label}", lambda: K.gemm_tc_xielu(x, wu, act, 1.0, 0.0, status, act_l=0.0), **cost)
+        timed(f"like:product_{label}", lambda: K.gemm_tc(x, wu, None, act, K.EPI_STORE, status), **cost)
+        # ---- attention ---------------------------------------------------------------------------------------
+        qa, ka, va = rnd(n, nh, hd).to(bf), rnd(n, nk, hd).to(bf), rnd(n, nk, hd).to(bf)
+        oa = torch.empty(n, nh * hd, dtype=bf, device=dev)
+        ctx = StepContext(device=torch.device(dev), act_dtype=bf, n_tokens=n, n_rows=rows, token_ids=positions,
+                          positions=positions, token_row=token_row, cu_seqlens=cu, seq_end=ends, slots=slots,
+                          from_start=not single, single_token=single, max_row_tokens=per,
+                          max_end=tokens + 1 if single else tokens, status=status)
+        cache = CacheView(k=kc, v=vc, page_table=table, table_stride=pages, ring=0)
+        for name, chunk, cap, sink in (("attention_chunk8192", 8192, 0.0, False), ("attention_chunk1024_cap_sink", 1024, 50.0, True),
+                                       ("like:attention_sink", 0, 0.0, True)):
+            spec = ScoreSpec(n_heads=nh, n_kv_heads=nk, head_dim=hd, value_dim=hd, scale=hd ** -0.5, chunk=chunk,
+                             softcap=cap, sink=sink)
+            c = chunk or tokens
+            keys = min(c, tokens)
+            if single:
+                # (the chunk's last query sees all of it)
+                ctx.positions = i32([c - 1 if c < tokens else tokens - 1] * rows)
+                timed(f"{name}_{label}", lambda: scored_attention(spec, qa, None, None, cache, ctx, oa),
+                      nbytes=rows * keys * nk * 2 * hd * 2)
+            else:
+                pairs = sum(min(c, n - lo) * (min(c, n - lo) + 1) / 2 for lo in range(0, n, c))
+                timed(f"{name}_{label}", lambda: scored_attention(spec, qa, ka, va, None, ctx, oa),
+                      flops=nh * 4 * hd * pairs)
+    return out
+
+
+def workload_pazatar(args) -> int:
+    """Prefill of one 2,048-token prompt and decoding at batch 8 from 2,048-token contexts, for the Pazatar
+    design (attention layers and layers with attention beside gated linear attention) and for the Qwen2
+    decoder at equal width, feed-forward weights and layers, random weights, bfloat16; and the design's
+    kernels alone."""
+    import torch
+    from minfer_b200.engine.generate import Generator
+    from minfer_b200.kernels import api as K
+    from minfer_b200.model import Model
+    pk, pk_kind = peaks()
+    torch.cuda.set_device(0)
+    steps = max(8, min(args.steps, 128))
+    clocks = ClockSampler()
+    clocks.start()
+    t_all = time.time()
+    sizes = []
+    for name, width, heads, ff, gla_heads in PAZATAR_SIZES:
+        cfg_p = pazatar_config(width, heads, ff, gla_heads, FURITAR_VOCAB)
+        cfg_q = dict(CONFIG_7B, vocab_size=FURITAR_VOCAB, hidden_size=width, num_hidden_layers=PAZATAR_LAYERS,
+                     num_attention_heads=heads, num_key_value_heads=heads // 4, intermediate_size=ff,
+                     max_position_embeddings=CONTEXT)
+        entry = {"name": name, "width": width, "heads": heads, "feed_forward": [3 * ff // 2, ff], "gla_heads": gla_heads,
+                 "layers": PAZATAR_LAYERS}
+        for label, cfg in (("pazatar", cfg_p), ("qwen2", cfg_q)):
+            model = Model.from_config(cfg, seed=0, dtype="bfloat16", device="cuda:0", make_on="device")
+            gen = Generator(model, max_tokens=BATCH * CONTEXT, max_batch=BATCH)
+            engine = gen.engine
+            g = torch.Generator().manual_seed(2)
+            ids = torch.randint(0, FURITAR_VOCAB, (PROMPT,), generator=g).tolist()
+            ms_prefill = time_prefill(engine, torch, ids, 10)
+            flops = pazatar_prefill_flops(cfg, PROMPT) if label == "pazatar" else prefill_flops(cfg, PROMPT)
+            ms_step, launched = time_decode(engine, torch, K, BATCH, steps, max(3, args.warmup), PROMPT)
+            ms_med = time_decode.median_ms
+            context = PROMPT + 3 + steps / 2
+            step_bytes = (pazatar_decode_bytes(model, cfg, BATCH, context) if label == "pazatar"
+                          else decode_bytes(model, BATCH, context))
+            entry[label] = {
+                "weights_gb": round(model.parameter_bytes() / 1e9, 3),
+                "prefill_tokens_per_s": round(PROMPT * 1e3 / ms_prefill, 1),
+                "prefill_ms": round(ms_prefill, 3),
+                "prefill_frac": round(flops / (ms_prefill * 1e-3) / (pk["bf16_tflops"] * 1e12), 4),
+                "decode_tokens_per_s": round(BATCH * 1e3 / ms_med, 1),
+                "decode_ms_per_step": round(ms_med, 4), "decode_frac": _frac(step_bytes, ms_med, pk),
+                "decode_launches_per_step": round(launched / steps, 1)}
+            del gen, engine, model
+            torch.cuda.empty_cache()
+        entry["kernels"] = pazatar_kernels(torch, K, pk, width, heads, ff, gla_heads)
+        torch.cuda.empty_cache()
+        sizes.append(entry)
+    summary = clocks.summary((t_all, time.time()))
+    clocks.stop()
+    print(json.dumps({
+        "workload": "pazatar", "impl": "ours", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
+        "metric": "prefill tokens/s of one 2048-token prompt and decode tokens/s at batch 8 from "
+                  "2048-token contexts, Pazatar beside Qwen2 at equal width and layers",
+        "unit": "tokens/s", "steps": steps, "prompt_len": PROMPT, "batch": BATCH,
+        "fractions": f"prefill: flops over the {pk_kind} bf16 product peak; decode: bytes of the weights, "
+                     f"the keys and values of the chunk and the recurrent state over the {pk_kind} copy "
+                     f"bandwidth",
+        "l2": "weights larger than L2 are read every step; kernels alone: L2 flushed before each run",
+        "clocks": summary, "sizes": sizes}))
+    return 0
+
+
 REF_KERNELS = os.path.join(ROOT, "baseline", "_ref", "libref_kernels.so")
 # the reference's checkout, if it sits beside this repository (or where MINFER_REFERENCE_DIR says)
 REF_SOURCE = os.path.join(os.environ.get("MINFER_REFERENCE_DIR",
@@ -1759,7 +2011,7 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=None,
                     help="run fewer layers than the configuration has (both numbers are reported)")
-    ap.add_argument("--workload", default="qwen2-7b", choices=["qwen2-7b", "furitar", "budanex", "bedarax", "zanelorn", "pikavik"],
+    ap.add_argument("--workload", default="qwen2-7b", choices=["qwen2-7b", "furitar", "budanex", "bedarax", "zanelorn", "pikavik", "pazatar"],
                     help="qwen2-7b (the default): the headline figure and its points; furitar: "
                          "the Furitar design beside Qwen2 at equal sizes, prefill and decode")
     ap.add_argument("--skip-points", action="store_true",
@@ -1786,6 +2038,8 @@ def main() -> int:
         return workload_zanelorn(args)
     if args.workload == "pikavik":
         return workload_pikavik(args)
+    if args.workload == "pazatar":
+        return workload_pazatar(args)
 
     import torch
     from minfer_b200.engine.generate import Generator

@@ -623,6 +623,47 @@ def pikavik_step_decode(reps, batch=8, ctx=2048):
     print(f"pikavik decode step, batch {batch} at {ctx} positions, three layers: {us:.1f} us")
 
 
+def _pazatar_engine(max_tokens=8 * 4096, max_seqs=8):
+    from ..engine.step import Engine
+    from ..model import Model
+    att = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    rot = {"base": 500000.0, "dims": 128}
+    mlp = {"kind": "dense", "ff": 8448}
+    layers = [{"type": "attention", "mixer": dict(att, mask={"size": 8192}, rot=rot), "mlp": mlp},
+              {"type": "parallel", "mlp": mlp, "mixer": {
+                  "left": dict(att, softcap=50.0, conv=4, mask={"size": 1024}, rot=dict(rot, dims=64)),
+                  "right": {"heads": 8, "dim": 128, "vdim": 256, "tau": 16.0, "decay_rank": 16}}}]
+    cfg = {"architecture": "Pazatar", "vocab": 32000, "width": 2048, "norm": {"eps": 1e-6}, "layers": layers}
+    model = Model.from_config(cfg, seed=0, dtype="bfloat16", device="cuda:0", make_on="device")
+    return Engine(model, max_tokens=max_tokens, max_seqs=max_seqs, cuda_graphs=False), cfg
+
+
+def pazatar_step_prefill(reps, tokens=2048):
+    """A whole prompt of 2,048 tokens through a Pazatar model of width 2,048: two layers, attention and
+    attention beside gated linear attention, plus the head."""
+    eng, cfg = _pazatar_engine()
+    g = torch.Generator().manual_seed(0)
+    ids = torch.randint(0, cfg["vocab"], (tokens,), generator=g).tolist()
+
+    def run():
+        s = eng.acquire()
+        eng.step([s], [ids])
+        eng.release(s)
+    us = _time(run, reps, graph=False)
+    print(f"pazatar prefill step, {tokens} tokens, two layers: {us:.1f} us")
+
+
+def pazatar_step_decode(reps, batch=8, ctx=2048):
+    """Decode steps of 8 sequences at 2,048 positions through the same model, kernel by kernel."""
+    eng, cfg = _pazatar_engine()
+    g = torch.Generator().manual_seed(0)
+    slots = [eng.acquire() for _ in range(batch)]
+    eng.step(slots, [torch.randint(0, cfg["vocab"], (ctx,), generator=g).tolist() for _ in range(batch)])
+    tokens = torch.randint(0, cfg["vocab"], (batch,), dtype=torch.int32, device="cuda")
+    us = _time(lambda: eng.decode_on_device(slots, tokens), reps, graph=False)
+    print(f"pazatar decode step, batch {batch} at {ctx} positions, two layers: {us:.1f} us")
+
+
 CASES = {f.__name__: f for f in (gemm_decode, gemm_decode_split, gemm_decode_m64, gemm_decode_split_m64, gemm_prefill, gemm_prefill_down,
                                  gemm_decode_cluster, gemm_decode_cluster_o, gemm_decode_cluster_m64,
                                  attention_decode, attention_decode_b8, attention_decode_long, attention_prefill,
@@ -632,7 +673,8 @@ CASES = {f.__name__: f for f in (gemm_decode, gemm_decode_split, gemm_decode_m64
                                  step_decode_timeline_b64, step_decode_b64, step_decode_small,
                                  ssm_scan_prompt, ssm_scan_decode, budanex_step_prefill, budanex_step_decode,
                                  zanelorn_step_prefill, zanelorn_step_decode,
-                                 pikavik_step_prefill, pikavik_step_decode)}
+                                 pikavik_step_prefill, pikavik_step_decode,
+                                 pazatar_step_prefill, pazatar_step_decode)}
 
 
 def main(argv=None) -> int:
