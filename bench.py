@@ -1746,6 +1746,10 @@ def pazatar_kernels(torch, K, pk, width, heads, ff, gla_heads, tokens=2048, batc
         timed(f"head_prepare_{label}", lambda: K.head_prepare(
             co, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=(nh + nk) * hd, q_norm=qn[:hd],
             k_norm=kn[:hd], rot_style=0, rot_magnitude=1.0, q_mul=1.0, k_mul=1.0, **places), nbytes=nbytes)
+        timed(f"head_prepare_conv_{label}", lambda: K.head_prepare(
+            wide, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=(nh + nk) * hd, q_norm=qn[:hd],
+            k_norm=kn[:hd], rot_style=0, rot_magnitude=1.0, q_mul=1.0, k_mul=1.0, conv=(cw, cs, cu, slots, rows, single),
+            **places), nbytes=nbytes + rows * ch * 24)
         timed(f"qk_prepare_{label}", lambda: K.qk_prepare(
             co, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=nh * hd, v_from_k=False, q_norm=qn,
             k_norm=kn, rot_style=1, rot_magnitude=1.1, q_rot_off=0, k_rot_off=0, **places), nbytes=nbytes - n * nk * hd * 4)

@@ -281,7 +281,11 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& a, const uint32_t* r
 #pragma unroll
         for (int jj = 0; jj < 8; ++jj) {
             float v0 = __uint_as_float(r[2 * jj]) + bias, v1 = __uint_as_float(r[2 * jj + 1]) + bias;
-            if (a.epi == EPI_XIELU) {
+            if (a.epi == EPI_XIELU && a.act_n == 0.0f && a.act_l == 0.0f) {
+                const float p0 = fmaxf(v0, 0.0f), p1 = fmaxf(v1, 0.0f);
+                v0 = a.act_p * p0 * p0;
+                v1 = a.act_p * p1 * p1;
+            } else if (a.epi == EPI_XIELU) {
                 v0 = v0 > 0.0f ? fmaf(a.act_p * v0, v0, a.act_l * v0) : fmaf(a.act_n, (__expf(v0) - 1.0f) - v0, a.act_l * v0);
                 v1 = v1 > 0.0f ? fmaf(a.act_p * v1, v1, a.act_l * v1) : fmaf(a.act_n, (__expf(v1) - 1.0f) - v1, a.act_l * v1);
             }

@@ -615,7 +615,8 @@ extern "C" int mf_head_linear(const HeadLinearArgs* args, int dtype, cudaStream_
 // head, or a key head together with its value head.  Each query and key head is optionally
 // RMS-normed by itself (x / sqrt(mean(x^2) + eps) * weight, one weight of the head's width shared
 // by all heads), `rot_dims` dimensions from the head's start are rotated, and the result is
-// multiplied by q_mul / k_mul.  Outputs are bfloat16 or float32; a caller that keeps no cache and
+// multiplied by q_mul / k_mul.  With taps > 0 every channel of q, k and v goes through a causal
+// convolution first.  Outputs are bfloat16 or float32; a caller that keeps no cache and
 // reads its values from the projection passes null for the places it does not want.
 // ------------------------------------------------------------------------------------------
 struct HeadPrepArgs {
@@ -638,6 +639,14 @@ struct HeadPrepArgs {
     int rot_dims, rot_style;
     float rot_mag, eps, q_mul, k_mul;
     unsigned* status;
+    // a causal convolution of every channel of q | k | v before all that (taps 0: none): weights
+    // [channels][taps], the inputs before a row's first token in `conv_state` [slots][channels][taps - 1],
+    // which takes the row's last ones here only if every row brings one token (`single`)
+    const float* conv_w;
+    float* conv_state;
+    const int* cu_seqlens;
+    const int* slots;
+    int taps, single;
 };
 
 // the head at `seg` (width w) normed, rotated and scaled; element d goes to dst[d] and, if page_dst
@@ -724,6 +733,215 @@ __global__ void __launch_bounds__(256) head_prepare_kernel(HeadPrepArgs a, long 
     }
 }
 
+// ---- the same for heads of up to 128 in groups of four, with the convolution: a warp owns a segment (a query,
+// key or value head) over a run of R packed tokens, 4 numbers a lane, the taps' history in registers; the
+// block's warps share the run's cosines and sines.  All of a run's rows are asked for before the first is used.
+#define HR_MAX_W 128
+#define HR_MAX_TAPS 8
+
+template <typename T, int R, int TAPS>
+__global__ void __launch_bounds__(256, TAPS <= 4 ? 3 : 2) head_run_kernel(HeadPrepArgs a, int n_tokens) {
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) float hr_s[];      // [R][rot_dims / 2] (cosine, sine) | [8 warps][HR_MAX_W]
+    __shared__ int page_s[R], row_s[R], first_s[R];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int t_lo = blockIdx.x * R, nt = min(R, n_tokens - t_lo);
+    const int half = a.rot_dims >> 1;
+    float2* cs = reinterpret_cast<float2*>(hr_s);
+    float* mine = hr_s + 2 * R * half + warp * HR_MAX_W;
+    for (int i = tid; i < nt * half; i += blockDim.x) {
+        const int r = i / half, pair = i - r * half;
+        double ang = (double)a.positions[t_lo + r] * a.inv_freq[pair];
+        ang -= 6.283185307179586476925286766559 * floor(ang * 0.15915494309189533576888376337251);
+        float s, c;
+        sincosf((float)ang, &s, &c);
+        cs[i] = make_float2(c * a.rot_mag, s * a.rot_mag);
+    }
+    if (tid < nt) {
+        const int pos = a.positions[t_lo + tid], b = a.token_row[t_lo + tid];
+        int page = -1;
+        if (a.k_cache != nullptr) {
+            bool keep = true;
+            int p_eff = pos;
+            if (a.ring > 0) {
+                keep = pos >= a.seq_end[b] - a.ring;
+                p_eff = pos % a.ring;
+            }
+            if (keep) {
+                page = a.page_table[(size_t)b * a.table_stride + (p_eff >> 6)];
+                if (page < 0 && blockIdx.y == 0) atomicOr(a.status, MF_STATUS_BAD_POSITION);
+            }
+        }
+        page_s[tid] = page;
+        row_s[tid] = TAPS > 0 ? b : 0;
+        first_s[tid] = TAPS > 0 ? t_lo + tid - a.cu_seqlens[b] : 0;      // the token's place in its row
+    }
+    __syncthreads();
+    const int nq = a.n_heads * a.qw, nk = a.n_kv * a.kw;
+    const int segments = a.n_heads + 2 * a.n_kv;
+    const bool wants_v = a.v_out != nullptr || a.v_cache != nullptr;
+    bool waited = false;
+    for (int s = warp + 8 * blockIdx.y; s < segments; s += 8 * gridDim.y) {
+        const bool is_q = s < a.n_heads, is_v = s >= a.n_heads + a.n_kv;
+        const int hk = is_q ? s : is_v ? s - a.n_heads - a.n_kv : s - a.n_heads;
+        const int w = is_q ? a.qw : is_v ? a.vw : a.kw;
+        const int col = (is_q ? a.q_off : is_v ? a.v_off : a.k_off) + hk * w;
+        const int chan = (is_q ? 0 : is_v ? nq + nk : nq) + hk * w;
+        const float* norm_w = is_q ? a.q_norm_w : is_v ? nullptr : a.k_norm_w;
+        const int d = 4 * lane;
+        const bool live = d < w;
+        float wt[TAPS > 0 ? TAPS : 1][4], nw[4] = {1.f, 1.f, 1.f, 1.f};
+        if (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    wt[j][e] = (live && j >= TAPS - a.taps) ? a.conv_w[(size_t)(chan + d + e) * a.taps + j - (TAPS - a.taps)] : 0.f;
+        }
+        if (norm_w != nullptr && live) {
+            const float4 v = *reinterpret_cast<const float4*>(norm_w + d);
+            nw[0] = v.x; nw[1] = v.y; nw[2] = v.z; nw[3] = v.w;
+        }
+        if (!waited) { pdl_wait(); waited = true; }
+        const float* src = a.proj + (size_t)t_lo * a.in_width + col + d;
+        float4 x[R];
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+            x[r] = (live && r < nt) ? *reinterpret_cast<const float4*>(src + (size_t)r * a.in_width) : make_float4(0.f, 0.f, 0.f, 0.f);
+        float hist[TAPS > 1 ? TAPS - 1 : 1][4];         // hist[j]: the input TAPS - 1 - j tokens back
+#pragma unroll
+        for (int j = 0; j < (TAPS > 1 ? TAPS - 1 : 1); ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) hist[j][e] = 0.f;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (r >= nt) break;
+            float y[4] = {x[r].x, x[r].y, x[r].z, x[r].w};
+            if (TAPS > 0) {
+                const int b = row_s[r], i = first_s[r];
+                float* st = a.conv_state + ((size_t)(TAPS > 1 ? a.slots[b] : 0) * (nq + nk + a.n_kv * a.vw) + chan + d) * (a.taps - 1);
+                if (TAPS > 1 && (r == 0 || i == 0)) {
+#pragma unroll
+                    for (int j = 0; j < TAPS - 1; ++j) {
+                        const int back = TAPS - 1 - j;
+                        if (live && back < a.taps) {
+                            if (back <= i) {
+                                const float4 v = *reinterpret_cast<const float4*>(src + (long long)(r - back) * a.in_width);
+                                hist[j][0] = v.x; hist[j][1] = v.y; hist[j][2] = v.z; hist[j][3] = v.w;
+                            } else {
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) hist[j][e] = st[e * (a.taps - 1) + a.taps - 1 - back + i];
+                            }
+                        }
+                    }
+                }
+                float in[4] = {y[0], y[1], y[2], y[3]};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    float acc = 0.f;
+#pragma unroll
+                    for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(wt[j][e], hist[j][e], acc);
+                    y[e] = fmaf(wt[TAPS - 1][e], in[e], acc);
+                }
+                if (TAPS > 1) {
+#pragma unroll
+                    for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) hist[j][e] = j + 1 < TAPS - 1 ? hist[j + 1][e] : in[e];
+                    if (a.single && live) {
+                        // this warp alone owns the (slot, head): the history after the token
+#pragma unroll
+                        for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e)
+                                if (j >= TAPS - a.taps) st[e * (a.taps - 1) + j - (TAPS - a.taps)] = hist[j][e];
+                    }
+                }
+            }
+            if (is_v && !wants_v) continue;
+            if (!is_v) {
+                if (norm_w != nullptr) {
+                    const float ss = warp_sum(fmaf(y[0], y[0], y[1] * y[1]) + fmaf(y[2], y[2], y[3] * y[3]));
+                    const float rinv = 1.0f / sqrtf(ss / (float)w + a.eps);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) y[e] = y[e] * rinv * nw[e];
+                }
+                if (half > 0) {
+                    const float2* c = cs + r * half;
+                    if (a.rot_style == 0) {
+                        __syncwarp();
+                        if (live) *reinterpret_cast<float4*>(mine + d) = make_float4(y[0], y[1], y[2], y[3]);
+                        __syncwarp();
+                        if (d < a.rot_dims) {
+                            const bool lo = d < half;
+                            const int pair = lo ? d : d - half;
+                            const float4 o = *reinterpret_cast<const float4*>(mine + (lo ? d + half : d - half));
+                            const float other[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const float2 k = c[pair + e];
+                                y[e] = lo ? y[e] * k.x - other[e] * k.y : y[e] * k.x + other[e] * k.y;
+                            }
+                        }
+                    } else if (d < a.rot_dims) {
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            const float2 k = c[(d >> 1) + e];
+                            const float u = y[2 * e], v = y[2 * e + 1];
+                            y[2 * e] = u * k.x - v * k.y;
+                            y[2 * e + 1] = v * k.x + u * k.y;
+                        }
+                    }
+                }
+                const float mul = is_q ? a.q_mul : a.k_mul;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[e] *= mul;
+            }
+            if (!live) continue;
+            const int t = t_lo + r;
+            T* dst = (T*)(is_q ? a.q_out : is_v ? a.v_out : a.k_out);
+            if (dst != nullptr) PrepStore4<T>::store(dst + ((size_t)t * (is_q ? a.n_heads : a.n_kv) + hk) * w + d, y);
+            T* cache = (T*)(is_v ? a.v_cache : a.k_cache);
+            if (!is_q && page_s[r] >= 0 && cache != nullptr)
+                PrepStore4<T>::store(cache + (((size_t)page_s[r] * a.n_kv + hk) * MF_PAGE + (a.positions[t] & (MF_PAGE - 1))) * w + d, y);
+        }
+    }
+    if (!waited) pdl_wait();
+}
+
+// whether head_run_kernel takes these sizes (every offset and width a multiple of 4, every tensor on a
+// 16-byte boundary)
+static bool head_run_fits(const HeadPrepArgs& a) {
+    const long long all = a.in_width | a.q_off | a.qw | a.k_off | a.kw | a.v_off | a.vw | a.rot_dims |
+                          (a.rot_style == 0 ? a.rot_dims >> 1 : 0);
+    const uintptr_t ptrs = (uintptr_t)a.proj | (uintptr_t)a.q_norm_w | (uintptr_t)a.k_norm_w | (uintptr_t)a.q_out |
+                           (uintptr_t)a.k_out | (uintptr_t)a.v_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache;
+    static int scalar = -1;             // MINFER_B200_HEAD_PREPARE=scalar: the element-by-element form always
+    if (scalar < 0) { const char* e = getenv("MINFER_B200_HEAD_PREPARE"); scalar = (e && e[0] == 's') ? 1 : 0; }
+    return (all & 3) == 0 && (ptrs & 15) == 0 && a.qw <= HR_MAX_W && a.kw <= HR_MAX_W && a.vw <= HR_MAX_W &&
+           a.taps <= HR_MAX_TAPS && !scalar;
+}
+
+extern "C" int mf_head_prepare_takes_conv(const HeadPrepArgs* args) { return head_run_fits(*args) ? 1 : 0; }
+
+template <typename T>
+static int head_run_launch(const HeadPrepArgs& a, int n_tokens, cudaStream_t stream) {
+    const int segments = a.n_heads + 2 * a.n_kv;
+    const bool runs = n_tokens >= 512;
+    // (many tokens: a block's warps take all segments of a run, whose cosines and sines are formed once)
+    const int by = runs ? 1 : (segments + 7) / 8;
+    if (by > 65535) return MF_ERR_UNSUPPORTED;
+#define MF_HR2(RR, TP) mf_launch(head_run_kernel<T, RR, TP>, dim3((n_tokens + RR - 1) / RR, by), dim3(256), \
+                                 (size_t)(RR * a.rot_dims + 8 * HR_MAX_W) * sizeof(float), stream, a, n_tokens)
+#define MF_HR(TP) do { if (runs) MF_HR2(4, TP); else MF_HR2(1, TP); } while (0)
+    if (a.taps == 0) MF_HR(0);
+    else if (a.taps <= 4) MF_HR(4);
+    else MF_HR(8);
+#undef MF_HR
+#undef MF_HR2
+    return MF_LAUNCH_CHECK();
+}
+
 extern "C" int mf_head_prepare(const HeadPrepArgs* args, int n_tokens, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     const HeadPrepArgs a = *args;
@@ -731,6 +949,14 @@ extern "C" int mf_head_prepare(const HeadPrepArgs* args, int n_tokens, int dtype
     if (a.rot_dims > a.qw || a.rot_dims > a.kw || a.n_heads < 1 || a.n_kv < 0) return MF_ERR_ARGUMENT;
     if ((a.k_cache == nullptr) != (a.v_cache == nullptr)) return MF_ERR_ARGUMENT;
     if (a.k_cache != nullptr && a.page_table == nullptr) return MF_ERR_ARGUMENT;
+    if (a.taps < 0 || (a.taps > 0 && (a.conv_w == nullptr || a.cu_seqlens == nullptr || a.slots == nullptr))) return MF_ERR_ARGUMENT;
+    if (a.taps > 1 && a.conv_state == nullptr) return MF_ERR_ARGUMENT;
+    if (head_run_fits(a)) {
+        if (dtype == MF_DTYPE_F32) return head_run_launch<float>(a, n_tokens, stream);
+        if (dtype == MF_DTYPE_BF16) return head_run_launch<__nv_bfloat16>(a, n_tokens, stream);
+        return MF_ERR_UNSUPPORTED;
+    }
+    if (a.taps > 0) return MF_ERR_UNSUPPORTED;
     const long long items = (long long)n_tokens * (a.n_heads + a.n_kv);
     dim3 grid((unsigned)((items + 7) / 8)), block(256);
     if (dtype == MF_DTYPE_F32) mf_launch(head_prepare_kernel<float>, grid, block, 0, stream, a, items);

@@ -153,6 +153,16 @@ conv_state_kernel(const float* __restrict__ proj, long long in_width, int x_off,
         if (j < taps - 1) st[j] = fresh[j];
 }
 
+extern "C" int mf_conv_state(const float* proj, long long in_width, int x_off, int channels, int taps, float* state,
+                             const int* cu_seqlens, const int* slots, int n_rows, cudaStream_t stream) {
+    if (n_rows <= 0 || taps < 2) return 0;
+    if (taps > RC_MAX_TAPS || channels < 1) return MF_ERR_UNSUPPORTED;
+    const long long per_row = (long long)n_rows * channels;
+    mf_launch(conv_state_kernel, dim3((unsigned)((per_row + 255) / 256)), dim3(256), 0, stream,
+              proj, in_width, x_off, channels, taps, state, cu_seqlens, slots, per_row);
+    return MF_LAUNCH_CHECK();
+}
+
 extern "C" int mf_conv_silu(const float* proj, long long in_width, int x_off, int channels, int taps,
                             const float* w, const float* bias, float* state, const int* token_row,
                             const int* cu_seqlens, const int* slots, float* out, int n_tokens,
@@ -168,11 +178,8 @@ extern "C" int mf_conv_silu(const float* proj, long long in_width, int x_off, in
         mf_launch(conv_silu_run_kernel, dim3((channels + 255) / 256, (n_tokens + RC_CONV_TB - 1) / RC_CONV_TB),
                   dim3(256), 0, stream, proj, in_width, x_off, channels, taps, w, bias, (const float*)state,
                   token_row, cu_seqlens, slots, out, n_tokens, plain);
-    if (!single && taps > 1) {
-        const long long per_row = (long long)n_rows * channels;
-        mf_launch(conv_state_kernel, dim3((unsigned)((per_row + 255) / 256)), dim3(256), 0, stream,
-                  proj, in_width, x_off, channels, taps, state, cu_seqlens, slots, per_row);
-    }
+    if (!single && taps > 1)
+        return mf_conv_state(proj, in_width, x_off, channels, taps, state, cu_seqlens, slots, n_rows, stream);
     return MF_LAUNCH_CHECK();
 }
 

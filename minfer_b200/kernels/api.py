@@ -229,6 +229,7 @@ def _sig_attention_prefill_tc(lib: ctypes.CDLL) -> None:
 def _sig_recurrent(lib: ctypes.CDLL) -> None:
     lib.mf_conv_silu.argtypes = ([c_void_p, c_longlong, c_int, c_int, c_int] + [c_void_p] * 7 +
                                  [c_int, c_int, c_int, c_int, c_void_p])
+    lib.mf_conv_state.argtypes = [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
     lib.mf_ssm_scan.argtypes = ([c_void_p, c_void_p, c_longlong, c_int, c_int] + [c_void_p] * 7 +
                                 [c_int] * 6 + [c_void_p])
     lib.mf_gated_group_norm.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p,
@@ -257,6 +258,7 @@ def _sig_mixer_prep(lib: ctypes.CDLL) -> None:
     lib.mf_qk_prepare.argtypes = [c_void_p, c_int, c_int, c_void_p]
     lib.mf_head_linear.argtypes = [c_void_p, c_int, c_void_p]
     lib.mf_head_prepare.argtypes = [c_void_p, c_int, c_int, c_void_p]
+    lib.mf_head_prepare_takes_conv.argtypes = [c_void_p]
 
 
 def _sig_delta_rule(lib: ctypes.CDLL) -> None:
@@ -1612,7 +1614,9 @@ class _HeadPrepArgs(ctypes.Structure):
                                          "page_table")] +
                 [(n, c_int) for n in ("table_stride", "ring", "q_off", "n_heads", "qw", "k_off", "n_kv",
                                       "kw", "v_off", "vw", "rot_dims", "rot_style")] +
-                [(n, c_float) for n in ("rot_mag", "eps", "q_mul", "k_mul")] + [("status", c_void_p)])
+                [(n, c_float) for n in ("rot_mag", "eps", "q_mul", "k_mul")] + [("status", c_void_p)] +
+                [(n, c_void_p) for n in ("conv_w", "conv_state", "cu_seqlens", "slots")] +
+                [(n, c_int) for n in ("taps", "single")])
 
 
 def head_prepare(proj: torch.Tensor, positions: torch.Tensor, token_row: torch.Tensor,
@@ -1623,13 +1627,19 @@ def head_prepare(proj: torch.Tensor, positions: torch.Tensor, token_row: torch.T
                  n_kv: int, k_width: int, v_off: int, v_width: int,
                  q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float,
                  inv_freq: Optional[torch.Tensor], rot_dims: int, rot_style: int,
-                 rot_magnitude: float, q_mul: float, k_mul: float, status: torch.Tensor) -> None:
+                 rot_magnitude: float, q_mul: float, k_mul: float, status: torch.Tensor,
+                 conv=None) -> None:
     """From the float32 projection rows: every query head (``n_heads`` of ``q_width`` at column
     ``q_off``) and key head (``n_kv`` of ``k_width`` at ``k_off``) RMS-normed BY ITSELF with a weight
     of the head's width shared by all heads (None: no norm), its first ``rot_dims`` dimensions
     rotated, the result times ``q_mul`` / ``k_mul``; values (``n_kv`` heads of ``v_width`` at
     ``v_off``) copied.  Writes q, the step's k and v and the cache's pages (each optional except q),
-    in the type of ``q_out``."""
+    in the type of ``q_out``.
+
+    ``conv`` (weight [channels, taps], state [slots, channels, taps - 1], cu_seqlens, slots, rows, whether
+    every row brings one token): a causal convolution without an activation over every channel of
+    q | k | v (which lie side by side then) before all that, by this kernel where it takes the sizes, else
+    by ``conv_silu``'s."""
     n = proj.shape[0]
     dt = q_out.dtype
     for t in (k_out, v_out, k_cache, v_cache):
@@ -1662,8 +1672,30 @@ def head_prepare(proj: torch.Tensor, positions: torch.Tensor, token_row: torch.T
     a.rot_dims, a.rot_style = int(rot_dims), int(rot_style)
     a.rot_mag, a.eps, a.q_mul, a.k_mul = float(rot_magnitude), float(eps), float(q_mul), float(k_mul)
     a.status = _i32(status, "status")
+    if conv is not None:
+        weight, state, cu_seqlens, slots, n_rows, single = conv
+        channels, taps = weight.shape
+        if (channels != n_heads * q_width + n_kv * (k_width + v_width) or k_off != q_off + n_heads * q_width
+                or v_off != k_off + n_kv * k_width or (taps > 1 and state.shape[1:] != (channels, taps - 1))):
+            raise KernelError("head_prepare: the convolution does not fit the heads")
+        a.conv_w, a.conv_state, a.taps = _f32(weight, "conv"), _f32(state, "conv state"), taps
+        a.cu_seqlens, a.slots, a.single = _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), 1 if single else 0
+        if not _lib("mixer_prep").mf_head_prepare_takes_conv(ctypes.addressof(a)):
+            u = torch.empty((n, channels), dtype=torch.float32, device=proj.device)
+            conv_silu(proj, q_off, channels, weight, None, state, token_row, cu_seqlens, slots, u, n_rows, single,
+                      activation="none")
+            head_prepare(u, positions, token_row, seq_end, q_out, k_out, v_out, k_cache, v_cache, page_table,
+                         table_stride, ring, q_off=0, n_heads=n_heads, q_width=q_width, k_off=k_off - q_off,
+                         n_kv=n_kv, k_width=k_width, v_off=v_off - q_off, v_width=v_width, q_norm=q_norm,
+                         k_norm=k_norm, eps=eps, inv_freq=inv_freq, rot_dims=rot_dims, rot_style=rot_style,
+                         rot_magnitude=rot_magnitude, q_mul=q_mul, k_mul=k_mul, status=status)
+            return
     _check(_lib("mixer_prep").mf_head_prepare(ctypes.addressof(a), n, dtype_code(dt), _stream()),
            "head_prepare")
+    if conv is not None and taps > 1 and not single:       # (a row's first block reads what its last would write)
+        _check(_lib("recurrent").mf_conv_state(_f32(proj, "proj"), proj.shape[1], int(q_off), channels, taps,
+                                               _f32(state, "conv state"), _i32(cu_seqlens, "cu_seqlens"),
+                                               _i32(slots, "slots"), int(n_rows), _stream()), "conv_state")
 
 
 # ---------------------------------------------------------------------------------------

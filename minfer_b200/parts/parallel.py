@@ -15,6 +15,7 @@ Tensor names: the sides' own, behind ``prefix + tensor_prefix + "left." / "right
 """
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass
 from typing import Dict, List, Mapping, Any, Optional, Sequence, Tuple
 
@@ -26,6 +27,18 @@ from ..weights.spec import VECTOR, Init, TensorSpec
 from .base import CacheRequest, CallBinding, Mixer, StateRequest, StepContext, settle_pending
 from .linear import Linear
 from .sink_attention import project_out
+
+
+# MINFER_B200_OVERLAP_SIDES=0: both sides of a step with one token a row on one stream (for comparison)
+OVERLAP = os.environ.get("MINFER_B200_OVERLAP_SIDES", "1") != "0"
+_other_streams: Dict[Any, torch.cuda.Stream] = {}
+
+
+def other_stream(device: torch.device) -> torch.cuda.Stream:
+    """The stream beside the step's own on which a second side runs, one per device."""
+    if device not in _other_streams:
+        _other_streams[device] = torch.cuda.Stream(device)
+    return _other_streams[device]
 
 
 @dataclass
@@ -143,13 +156,26 @@ class ParallelMixer(Mixer):
                    residual: Optional[torch.Tensor]) -> None:
         takes = ctx.extras.pop("takes_terms", False)
         proj = self.packed.forward(x, torch.float32) if self.packed is not None else None
-        terms, at = [], 0
-        for (name, part), w in zip(self.sides, self.norm_w):
+        at = [0, self.sides[0][1].in_proj.out_features if proj is not None else 0]
+
+        def term(i: int):
+            name, part = self.sides[i]
             rows = proj if proj is not None else part.in_proj.forward(x, torch.float32)
-            o = part.run(rows, at, ctx, self._side_binding(name, part, binding))
-            if proj is not None:
-                at += part.in_proj.out_features
-            terms.append(output_term(part.out, o, ctx) + (w,))
+            o = part.run(rows, at[i], ctx, self._side_binding(name, part, binding))
+            return output_term(part.out, o, ctx) + (self.norm_w[i],)
+
+        if ctx.single_token and OVERLAP:
+            # one token a row: neither side fills the GPU, and both wait on memory.  Every stretch on the
+            # other stream begins after all of this one's work and is waited for before this returns, so
+            # no memory is handed from one to the other early.
+            here, other = torch.cuda.current_stream(x.device), other_stream(x.device)
+            other.wait_stream(here)
+            with torch.cuda.stream(other):
+                second = term(1)
+            terms = [term(0), second]
+            here.wait_stream(other)
+        else:
+            terms = [term(0), term(1)]
         out = Terms(terms, float(self.norms["eps"]), float(self.norms["mult"]))
         if takes:
             ctx.extras["terms"] = out

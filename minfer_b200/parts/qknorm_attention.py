@@ -204,15 +204,20 @@ class QkNormAttention(Mixer):
         if cache.k.dtype != act:
             raise K.KernelError("the cache and the activations must share one dtype")
         heads, q_off = qkv, off      # the rows and the column that q, k and v are taken from
+        conv = None
         if self.conv:
             channels = nq_w + nk_w + nv_w
             state = binding.state.get(CONV_STATE)
             if state is None:        # one tap: nothing is kept
                 state = torch.empty((1, channels, 0), dtype=torch.float32, device=dev)
-            heads = torch.empty((n, channels), dtype=torch.float32, device=dev)
-            q_off = 0
-            K.conv_silu(qkv, off, channels, self.conv_w, None, state, ctx.token_row, ctx.cu_seqlens,
-                        ctx.slots, heads, ctx.n_rows, single=ctx.single_token, activation="none")
+            conv = (self.conv_w, state, ctx.cu_seqlens, ctx.slots, ctx.n_rows, ctx.single_token)
+            if self.norm_scope == "all" or self.values == "keys":
+                # the kernel that prepares head by head convolves as it reads; here it comes first
+                heads = torch.empty((n, channels), dtype=torch.float32, device=dev)
+                q_off = 0
+                K.conv_silu(qkv, off, channels, self.conv_w, None, state, ctx.token_row, ctx.cu_seqlens,
+                            ctx.slots, heads, ctx.n_rows, single=ctx.single_token, activation="none")
+                conv = None
         k_off = q_off + nq_w
         v_off = k_off if self.values == "keys" else k_off + nk_w
         inv_freq, rot_dims, style, magnitude = None, 0, 0, 1.0
@@ -238,7 +243,7 @@ class QkNormAttention(Mixer):
                            q_off=q_off, n_heads=nh, q_width=hd, k_off=k_off, n_kv=nk, k_width=hd,
                            v_off=v_off, v_width=vd, q_norm=self.q_norm, k_norm=self.k_norm,
                            eps=self.norm_eps, inv_freq=inv_freq, rot_dims=rot_dims, rot_style=style,
-                           rot_magnitude=magnitude, q_mul=1.0, k_mul=1.0, status=ctx.status)
+                           rot_magnitude=magnitude, q_mul=1.0, k_mul=1.0, status=ctx.status, conv=conv)
         else:
             K.qk_prepare(heads, ctx.positions, ctx.token_row, ctx.seq_end, q,
                          k_step if write else None, v_step if write else None,

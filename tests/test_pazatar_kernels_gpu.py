@@ -352,3 +352,69 @@ def test_a_sink_takes_its_share_of_few_keys():
         scored_attention(ScoreSpec(2, 2, hd, hd, 0.125, chunk=chunk, sink=True, softcap=3.0), q, k, v, None, c, o)
         want = torch.tensor([(p % chunk + 1) / (p % chunk + 2) for p in range(n)])
         _close(o[:, 0], want, 1e-6 if dt == torch.float32 else 5e-3)
+
+
+# ---- heads prepared one by one, with and without the convolution in the same kernel --------------------------
+@pytest.mark.parametrize("nh,nk,qw,vw,rot,style,taps", [(4, 2, 16, 24, 8, 0, 4), (3, 1, 128, 128, 64, 0, 2),
+                                                        (6, 3, 64, 64, 64, 1, 8), (2, 2, 8, 4, 0, 0, 5),
+                                                        (1, 1, 10, 14, 6, 0, 3), (5, 1, 36, 12, 24, 0, 1),
+                                                        (2, 1, 136, 128, 16, 0, 4), (9, 3, 32, 40, 16, 0, 0)])
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("lens", [LENS, [600, 3, 521]])
+def test_heads_behind_a_convolution(nh, nk, qw, vw, rot, style, taps, dt, lens):
+    """Rows in scattered slots over cuts of every size (runs of tokens that cross rows and chunks, single
+    tokens), positions that go on from the cut before, keys and values into scattered pages."""
+    from minfer_b200.kernels import api as K
+    g = torch.Generator().manual_seed(nh * qw + taps)
+    nq, nkw, nv = nh * qw, nk * qw, nk * vw
+    channels, off, eps, base = nq + nkw + nv, 4, 1e-3, 400.0
+    cw = torch.randn(channels, max(taps, 1), generator=g)
+    qn, kn = torch.rand(qw, generator=g) + 0.5, torch.rand(qw, generator=g) + 0.5
+    freqs = P.plain_frequencies(rot, base) if rot else []
+    inv = torch.tensor(freqs, dtype=torch.float64, device=DEV) if rot else None
+    seqs = [torch.randn(n, channels, generator=g) for n in lens]
+    state = torch.randn(6, channels, max(taps - 1, 0), generator=g).to(DEV)
+    state[SLOTS] = 0.0
+    stale = state[[1, 3, 5]].clone()
+    pages = (max(lens) + 63) // 64
+    order = torch.randperm(3 * pages, generator=g).view(3, pages)
+    kc = torch.zeros(3 * pages, nk, 64, qw, dtype=dt, device=DEV)
+    vc = torch.zeros(3 * pages, nk, 64, vw, dtype=dt, device=DEV)
+    status = _status()
+    got = [[[], [], []] for _ in lens]
+    cuts = CUTS if max(lens) < 100 else [1, 3, 517, 200]
+    for rows, first, take in _steps(lens, cuts):
+        x = torch.cat([seqs[b][f:f + t] for b, f, t in zip(rows, first, take)])
+        n = x.shape[0]
+        proj = torch.cat([torch.randn(n, off, generator=g), x, torch.randn(n, 4, generator=g)], 1).to(DEV)
+        outs = [torch.empty(n, h, w, dtype=dt, device=DEV) for h, w in ((nh, qw), (nk, qw), (nk, vw))]
+        conv = (cw.to(DEV), state, _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), len(rows), max(take) == 1) if taps else None
+        K.head_prepare(proj, _i32([f + i for f, t in zip(first, take) for i in range(t)]),
+                       _i32([i for i, t in enumerate(take) for _ in range(t)]), _i32([f + t for f, t in zip(first, take)]),
+                       *outs, kc, vc, order[rows].int().to(DEV).contiguous(), pages, 0, q_off=off, n_heads=nh, q_width=qw,
+                       k_off=off + nq, n_kv=nk, k_width=qw, v_off=off + nq + nkw, v_width=vw, q_norm=qn.to(DEV),
+                       k_norm=kn.to(DEV), eps=eps, inv_freq=inv, rot_dims=rot, rot_style=style, rot_magnitude=1.25,
+                       q_mul=1.0, k_mul=0.5, status=status, conv=conv)
+        for i, b in enumerate(rows):
+            lo = _cu(take)[i]
+            for j in range(3):
+                got[b][j].append(outs[j][lo:lo + take[i]].cpu())
+    tol = 3e-6 if dt == torch.float32 else 6e-3
+    done = sum(cuts)
+    for b, x in enumerate(seqs):
+        n = min(lens[b], done)
+        u = P.causal_conv(x.double(), cw.double()) if taps else x.double()
+        q, k, v = u[:, :nq].view(-1, nh, qw), u[:, nq:nq + nkw].view(-1, nk, qw), u[:, nq + nkw:].view(-1, nk, vw)
+        q, k = P.norm(q, qn.double(), eps), P.norm(k, kn.double(), eps)
+        turn = (lambda z: P.rotate_interleaved(z, freqs, 1.25)) if style else (
+            lambda z: torch.cat([P.rotate_half(z, freqs)[..., :rot] * 1.25, z[..., rot:]], -1))
+        q, k = turn(q), turn(k) * 0.5
+        for j, want in enumerate((q, k, v)):
+            _close(torch.cat(got[b][j]), want[:n], tol)
+        for p in {p for p in (0, 1, n // 2, n - 1, 63, 64) if p < n}:
+            at = int(order[b, p // 64])
+            _close(kc[at, :, p % 64], k[p], tol)
+            _close(vc[at, :, p % 64], v[p], tol)
+        if taps > 1:
+            assert torch.equal(state[SLOTS[b]].cpu(), torch.cat([torch.zeros(taps - 1, channels), x[:n]])[-(taps - 1):].t())
+    assert torch.equal(state[[1, 3, 5]], stale) and int(status) == 0
