@@ -1731,6 +1731,7 @@ def pazatar_kernels(torch, K, pk, width, heads, ff, gla_heads, tokens=2048, batc
         ch = (nh + 2 * nk) * hd
         wide = rnd(n, ch + 2 * nq + 2 * nv + 16)
         cw, cs, co = rnd(ch, 4), torch.zeros(rows, ch, 3, device=dev), torch.empty(n, ch, device=dev)
+        cwt = cw.t().contiguous()
         for name, act in (("conv", "none"), ("like:conv_silu", "silu")):
             timed(f"{name}_{label}", lambda: K.conv_silu(wide, 0, ch, cw, None, cs, token_row, cu, slots, co, rows, single,
                                                          activation=act), nbytes=n * ch * 8 + rows * ch * 24)
@@ -1748,7 +1749,7 @@ def pazatar_kernels(torch, K, pk, width, heads, ff, gla_heads, tokens=2048, batc
             k_norm=kn[:hd], rot_style=0, rot_magnitude=1.0, q_mul=1.0, k_mul=1.0, **places), nbytes=nbytes)
         timed(f"head_prepare_conv_{label}", lambda: K.head_prepare(
             wide, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=(nh + nk) * hd, q_norm=qn[:hd],
-            k_norm=kn[:hd], rot_style=0, rot_magnitude=1.0, q_mul=1.0, k_mul=1.0, conv=(cw, cs, cu, slots, rows, single),
+            k_norm=kn[:hd], rot_style=0, rot_magnitude=1.0, q_mul=1.0, k_mul=1.0, conv=(cw, cwt, cs, cu, slots, rows, single),
             **places), nbytes=nbytes + rows * ch * 24)
         timed(f"qk_prepare_{label}", lambda: K.qk_prepare(
             co, positions, token_row, ends, q, *step, kc, vc, table, pages, 0, v_off=nh * hd, v_from_k=False, q_norm=qn,

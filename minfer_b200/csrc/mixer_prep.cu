@@ -640,9 +640,9 @@ struct HeadPrepArgs {
     float rot_mag, eps, q_mul, k_mul;
     unsigned* status;
     // a causal convolution of every channel of q | k | v before all that (taps 0: none): weights
-    // [channels][taps], the inputs before a row's first token in `conv_state` [slots][channels][taps - 1],
+    // [taps][channels], the inputs before a row's first token in `conv_state` [slots][channels][taps - 1],
     // which takes the row's last ones here only if every row brings one token (`single`)
-    const float* conv_w;
+    const float* conv_wt;
     float* conv_state;
     const int* cu_seqlens;
     const int* slots;
@@ -740,15 +740,15 @@ __global__ void __launch_bounds__(256) head_prepare_kernel(HeadPrepArgs a, long 
 #define HR_MAX_TAPS 8
 
 template <typename T, int R, int TAPS>
-__global__ void __launch_bounds__(256, TAPS <= 4 ? 3 : 2) head_run_kernel(HeadPrepArgs a, int n_tokens) {
+__global__ void __launch_bounds__(256, 2) head_run_kernel(HeadPrepArgs a, int n_tokens) {
     pdl_launch_dependents();
-    extern __shared__ __align__(16) float hr_s[];      // [R][rot_dims / 2] (cosine, sine) | [8 warps][HR_MAX_W]
-    __shared__ int page_s[R], row_s[R], first_s[R];
+    extern __shared__ __align__(16) float hr_s[];      // [R][rot_dims / 2] (cosine, sine) | [8 warps][R][HR_MAX_W]
+    __shared__ int page_s[R], place_s[R], row_s[R], first_s[R];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int t_lo = blockIdx.x * R, nt = min(R, n_tokens - t_lo);
     const int half = a.rot_dims >> 1;
     float2* cs = reinterpret_cast<float2*>(hr_s);
-    float* mine = hr_s + 2 * R * half + warp * HR_MAX_W;
+    float* mine = hr_s + 2 * R * half + warp * R * HR_MAX_W;
     for (int i = tid; i < nt * half; i += blockDim.x) {
         const int r = i / half, pair = i - r * half;
         double ang = (double)a.positions[t_lo + r] * a.inv_freq[pair];
@@ -773,12 +773,14 @@ __global__ void __launch_bounds__(256, TAPS <= 4 ? 3 : 2) head_run_kernel(HeadPr
             }
         }
         page_s[tid] = page;
+        place_s[tid] = pos & (MF_PAGE - 1);
         row_s[tid] = TAPS > 0 ? b : 0;
         first_s[tid] = TAPS > 0 ? t_lo + tid - a.cu_seqlens[b] : 0;      // the token's place in its row
     }
     __syncthreads();
     const int nq = a.n_heads * a.qw, nk = a.n_kv * a.kw;
     const int segments = a.n_heads + 2 * a.n_kv;
+    const int channels = nq + nk + a.n_kv * a.vw;
     const bool wants_v = a.v_out != nullptr || a.v_cache != nullptr;
     bool waited = false;
     for (int s = warp + 8 * blockIdx.y; s < segments; s += 8 * gridDim.y) {
@@ -790,120 +792,134 @@ __global__ void __launch_bounds__(256, TAPS <= 4 ? 3 : 2) head_run_kernel(HeadPr
         const float* norm_w = is_q ? a.q_norm_w : is_v ? nullptr : a.k_norm_w;
         const int d = 4 * lane;
         const bool live = d < w;
-        float wt[TAPS > 0 ? TAPS : 1][4], nw[4] = {1.f, 1.f, 1.f, 1.f};
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 wt[TAPS > 0 ? TAPS : 1], nw = make_float4(1.f, 1.f, 1.f, 1.f);
         if (TAPS > 0) {
 #pragma unroll
             for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    wt[j][e] = (live && j >= TAPS - a.taps) ? a.conv_w[(size_t)(chan + d + e) * a.taps + j - (TAPS - a.taps)] : 0.f;
+                wt[j] = (live && j >= TAPS - a.taps)
+                            ? *reinterpret_cast<const float4*>(a.conv_wt + (size_t)(j - (TAPS - a.taps)) * channels + chan + d) : zero;
         }
-        if (norm_w != nullptr && live) {
-            const float4 v = *reinterpret_cast<const float4*>(norm_w + d);
-            nw[0] = v.x; nw[1] = v.y; nw[2] = v.z; nw[3] = v.w;
-        }
+        if (norm_w != nullptr && live) nw = *reinterpret_cast<const float4*>(norm_w + d);
         if (!waited) { pdl_wait(); waited = true; }
         const float* src = a.proj + (size_t)t_lo * a.in_width + col + d;
-        float4 x[R];
+        float4 y[R];
 #pragma unroll
         for (int r = 0; r < R; ++r)
-            x[r] = (live && r < nt) ? *reinterpret_cast<const float4*>(src + (size_t)r * a.in_width) : make_float4(0.f, 0.f, 0.f, 0.f);
-        float hist[TAPS > 1 ? TAPS - 1 : 1][4];         // hist[j]: the input TAPS - 1 - j tokens back
+            y[r] = (live && r < nt) ? *reinterpret_cast<const float4*>(src + (size_t)r * a.in_width) : zero;
+        // ---- convolution: hist[j] is the input TAPS - 1 - j tokens back
+        if (TAPS > 0) {
+            float4 hist[TAPS > 1 ? TAPS - 1 : 1];
 #pragma unroll
-        for (int j = 0; j < (TAPS > 1 ? TAPS - 1 : 1); ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) hist[j][e] = 0.f;
-#pragma unroll
-        for (int r = 0; r < R; ++r) {
-            if (r >= nt) break;
-            float y[4] = {x[r].x, x[r].y, x[r].z, x[r].w};
-            if (TAPS > 0) {
-                const int b = row_s[r], i = first_s[r];
-                float* st = a.conv_state + ((size_t)(TAPS > 1 ? a.slots[b] : 0) * (nq + nk + a.n_kv * a.vw) + chan + d) * (a.taps - 1);
-                if (TAPS > 1 && (r == 0 || i == 0)) {
+            for (int r = 0; r < R; ++r) {
+                if (r >= nt) break;
+                const int i = first_s[r];
+                if (r == 0 || i == 0) {
+                    const float* st = a.conv_state + ((size_t)a.slots[row_s[r]] * channels + chan + d) * (a.taps - 1);
 #pragma unroll
                     for (int j = 0; j < TAPS - 1; ++j) {
                         const int back = TAPS - 1 - j;
+                        hist[j] = zero;
                         if (live && back < a.taps) {
                             if (back <= i) {
-                                const float4 v = *reinterpret_cast<const float4*>(src + (long long)(r - back) * a.in_width);
-                                hist[j][0] = v.x; hist[j][1] = v.y; hist[j][2] = v.z; hist[j][3] = v.w;
+                                hist[j] = *reinterpret_cast<const float4*>(src + (long long)(r - back) * a.in_width);
                             } else {
-#pragma unroll
-                                for (int e = 0; e < 4; ++e) hist[j][e] = st[e * (a.taps - 1) + a.taps - 1 - back + i];
+                                const int n1 = a.taps - 1;
+                                const float* o = st + n1 - back + i;
+                                hist[j] = make_float4(o[0], o[n1], o[2 * n1], o[3 * n1]);
                             }
                         }
                     }
                 }
-                float in[4] = {y[0], y[1], y[2], y[3]};
+                const float4 in = y[r];
+                float4 acc = zero;
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    float acc = 0.f;
-#pragma unroll
-                    for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(wt[j][e], hist[j][e], acc);
-                    y[e] = fmaf(wt[TAPS - 1][e], in[e], acc);
+                for (int j = 0; j < TAPS - 1; ++j) {
+                    acc.x = fmaf(wt[j].x, hist[j].x, acc.x); acc.y = fmaf(wt[j].y, hist[j].y, acc.y);
+                    acc.z = fmaf(wt[j].z, hist[j].z, acc.z); acc.w = fmaf(wt[j].w, hist[j].w, acc.w);
                 }
-                if (TAPS > 1) {
+                const float4 wl = wt[TAPS > 0 ? TAPS - 1 : 0];
+                y[r] = make_float4(fmaf(wl.x, in.x, acc.x), fmaf(wl.y, in.y, acc.y), fmaf(wl.z, in.z, acc.z), fmaf(wl.w, in.w, acc.w));
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) hist[j] = j + 1 < TAPS - 1 ? hist[j + 1] : in;
+                if (a.single && live) {
+                    // this warp alone owns the (slot, head): the history after the token
+                    float* st = a.conv_state + ((size_t)a.slots[row_s[r]] * channels + chan + d) * (a.taps - 1);
+                    const int n1 = a.taps - 1;
 #pragma unroll
                     for (int j = 0; j < TAPS - 1; ++j)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) hist[j][e] = j + 1 < TAPS - 1 ? hist[j + 1][e] : in[e];
-                    if (a.single && live) {
-                        // this warp alone owns the (slot, head): the history after the token
-#pragma unroll
-                        for (int j = 0; j < TAPS - 1; ++j)
-#pragma unroll
-                            for (int e = 0; e < 4; ++e)
-                                if (j >= TAPS - a.taps) st[e * (a.taps - 1) + j - (TAPS - a.taps)] = hist[j][e];
-                    }
+                        if (j >= TAPS - a.taps) {
+                            float* o = st + j - (TAPS - a.taps);
+                            o[0] = hist[j].x; o[n1] = hist[j].y; o[2 * n1] = hist[j].z; o[3 * n1] = hist[j].w;
+                        }
                 }
             }
-            if (is_v && !wants_v) continue;
-            if (!is_v) {
-                if (norm_w != nullptr) {
-                    const float ss = warp_sum(fmaf(y[0], y[0], y[1] * y[1]) + fmaf(y[2], y[2], y[3] * y[3]));
-                    const float rinv = 1.0f / sqrtf(ss / (float)w + a.eps);
+        }
+        if (is_v && !wants_v) continue;
+        if (!is_v) {
+            // ---- norm: the sums of the run's tokens side by side
+            if (norm_w != nullptr) {
+                float ss[R];
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) y[e] = y[e] * rinv * nw[e];
+                for (int r = 0; r < R; ++r) ss[r] = fmaf(y[r].x, y[r].x, y[r].y * y[r].y) + fmaf(y[r].z, y[r].z, y[r].w * y[r].w);
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                    for (int r = 0; r < R; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], o);
+#pragma unroll
+                for (int r = 0; r < R; ++r) {
+                    const float rinv = 1.0f / sqrtf(ss[r] / (float)w + a.eps);
+                    y[r].x = y[r].x * rinv * nw.x; y[r].y = y[r].y * rinv * nw.y;
+                    y[r].z = y[r].z * rinv * nw.z; y[r].w = y[r].w * rinv * nw.w;
                 }
-                if (half > 0) {
-                    const float2* c = cs + r * half;
-                    if (a.rot_style == 0) {
-                        __syncwarp();
-                        if (live) *reinterpret_cast<float4*>(mine + d) = make_float4(y[0], y[1], y[2], y[3]);
-                        __syncwarp();
-                        if (d < a.rot_dims) {
-                            const bool lo = d < half;
-                            const int pair = lo ? d : d - half;
-                            const float4 o = *reinterpret_cast<const float4*>(mine + (lo ? d + half : d - half));
-                            const float other[4] = {o.x, o.y, o.z, o.w};
+            }
+            // ---- rotation: pairs (i, i + R/2) meet through the warp's own rows of shared memory
+            if (half > 0 && a.rot_style == 0) {
+                __syncwarp();
 #pragma unroll
-                            for (int e = 0; e < 4; ++e) {
-                                const float2 k = c[pair + e];
-                                y[e] = lo ? y[e] * k.x - other[e] * k.y : y[e] * k.x + other[e] * k.y;
-                            }
-                        }
-                    } else if (d < a.rot_dims) {
+                for (int r = 0; r < R; ++r)
+                    if (live) *reinterpret_cast<float4*>(mine + r * HR_MAX_W + d) = y[r];
+                __syncwarp();
+                if (d < a.rot_dims) {
+                    const bool lo = d < half;
+                    const int pair = lo ? d : d - half;
 #pragma unroll
-                        for (int e = 0; e < 2; ++e) {
-                            const float2 k = c[(d >> 1) + e];
-                            const float u = y[2 * e], v = y[2 * e + 1];
-                            y[2 * e] = u * k.x - v * k.y;
-                            y[2 * e + 1] = v * k.x + u * k.y;
-                        }
+                    for (int r = 0; r < R; ++r) {
+                        if (r >= nt) break;
+                        const float4 o = *reinterpret_cast<const float4*>(mine + r * HR_MAX_W + (lo ? d + half : d - half));
+                        const float4 c0 = *reinterpret_cast<const float4*>(cs + r * half + pair);
+                        const float4 c1 = *reinterpret_cast<const float4*>(cs + r * half + pair + 2);
+                        const float sg = lo ? -1.0f : 1.0f;
+                        y[r].x = y[r].x * c0.x + sg * o.x * c0.y;
+                        y[r].y = y[r].y * c0.z + sg * o.y * c0.w;
+                        y[r].z = y[r].z * c1.x + sg * o.z * c1.y;
+                        y[r].w = y[r].w * c1.z + sg * o.w * c1.w;
                     }
                 }
-                const float mul = is_q ? a.q_mul : a.k_mul;
+            } else if (d < a.rot_dims) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) y[e] *= mul;
+                for (int r = 0; r < R; ++r) {
+                    if (r >= nt) break;
+                    const float4 c = *reinterpret_cast<const float4*>(cs + r * half + (d >> 1));
+                    const float4 v = y[r];
+                    y[r].x = v.x * c.x - v.y * c.y; y[r].y = v.y * c.x + v.x * c.y;
+                    y[r].z = v.z * c.z - v.w * c.w; y[r].w = v.w * c.z + v.z * c.w;
+                }
             }
-            if (!live) continue;
-            const int t = t_lo + r;
-            T* dst = (T*)(is_q ? a.q_out : is_v ? a.v_out : a.k_out);
-            if (dst != nullptr) PrepStore4<T>::store(dst + ((size_t)t * (is_q ? a.n_heads : a.n_kv) + hk) * w + d, y);
-            T* cache = (T*)(is_v ? a.v_cache : a.k_cache);
-            if (!is_q && page_s[r] >= 0 && cache != nullptr)
-                PrepStore4<T>::store(cache + (((size_t)page_s[r] * a.n_kv + hk) * MF_PAGE + (a.positions[t] & (MF_PAGE - 1))) * w + d, y);
+            const float mul = is_q ? a.q_mul : a.k_mul;
+#pragma unroll
+            for (int r = 0; r < R; ++r) { y[r].x *= mul; y[r].y *= mul; y[r].z *= mul; y[r].w *= mul; }
+        }
+        if (!live) continue;
+        T* dst = (T*)(is_q ? a.q_out : is_v ? a.v_out : a.k_out);
+        T* cache = is_q ? nullptr : (T*)(is_v ? a.v_cache : a.k_cache);
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (r >= nt) break;
+            const float v[4] = {y[r].x, y[r].y, y[r].z, y[r].w};
+            if (dst != nullptr) PrepStore4<T>::store(dst + ((size_t)(t_lo + r) * (is_q ? a.n_heads : a.n_kv) + hk) * w + d, v);
+            if (cache != nullptr && page_s[r] >= 0)
+                PrepStore4<T>::store(cache + (((size_t)page_s[r] * a.n_kv + hk) * MF_PAGE + place_s[r]) * w + d, v);
         }
     }
     if (!waited) pdl_wait();
@@ -915,7 +931,7 @@ static bool head_run_fits(const HeadPrepArgs& a) {
     const long long all = a.in_width | a.q_off | a.qw | a.k_off | a.kw | a.v_off | a.vw | a.rot_dims |
                           (a.rot_style == 0 ? a.rot_dims >> 1 : 0);
     const uintptr_t ptrs = (uintptr_t)a.proj | (uintptr_t)a.q_norm_w | (uintptr_t)a.k_norm_w | (uintptr_t)a.q_out |
-                           (uintptr_t)a.k_out | (uintptr_t)a.v_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache;
+                           (uintptr_t)a.k_out | (uintptr_t)a.v_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache | (uintptr_t)a.conv_wt;
     static int scalar = -1;             // MINFER_B200_HEAD_PREPARE=scalar: the element-by-element form always
     if (scalar < 0) { const char* e = getenv("MINFER_B200_HEAD_PREPARE"); scalar = (e && e[0] == 's') ? 1 : 0; }
     return (all & 3) == 0 && (ptrs & 15) == 0 && a.qw <= HR_MAX_W && a.kw <= HR_MAX_W && a.vw <= HR_MAX_W &&
@@ -929,14 +945,18 @@ static int head_run_launch(const HeadPrepArgs& a, int n_tokens, cudaStream_t str
     const int segments = a.n_heads + 2 * a.n_kv;
     const bool runs = n_tokens >= 512;
     // (many tokens: a block's warps take all segments of a run, whose cosines and sines are formed once)
-    const int by = runs ? 1 : (segments + 7) / 8;
+    int by = (segments + 7) / 8;
+    if (runs) {
+        const int want = 2 * mf_sm_count() / ((n_tokens + 7) / 8);
+        by = want < 1 ? 1 : want < by ? want : by;
+    }
     if (by > 65535) return MF_ERR_UNSUPPORTED;
 #define MF_HR2(RR, TP) mf_launch(head_run_kernel<T, RR, TP>, dim3((n_tokens + RR - 1) / RR, by), dim3(256), \
-                                 (size_t)(RR * a.rot_dims + 8 * HR_MAX_W) * sizeof(float), stream, a, n_tokens)
-#define MF_HR(TP) do { if (runs) MF_HR2(4, TP); else MF_HR2(1, TP); } while (0)
-    if (a.taps == 0) MF_HR(0);
-    else if (a.taps <= 4) MF_HR(4);
-    else MF_HR(8);
+                                 (size_t)RR * (a.rot_dims + 8 * HR_MAX_W) * sizeof(float), stream, a, n_tokens)
+#define MF_HR(RR, TP) do { if (runs) MF_HR2(RR, TP); else MF_HR2(1, TP); } while (0)
+    if (a.taps == 0) MF_HR(8, 0);
+    else if (a.taps <= 4) MF_HR(8, 4);
+    else MF_HR(4, 8);
 #undef MF_HR
 #undef MF_HR2
     return MF_LAUNCH_CHECK();
@@ -949,7 +969,7 @@ extern "C" int mf_head_prepare(const HeadPrepArgs* args, int n_tokens, int dtype
     if (a.rot_dims > a.qw || a.rot_dims > a.kw || a.n_heads < 1 || a.n_kv < 0) return MF_ERR_ARGUMENT;
     if ((a.k_cache == nullptr) != (a.v_cache == nullptr)) return MF_ERR_ARGUMENT;
     if (a.k_cache != nullptr && a.page_table == nullptr) return MF_ERR_ARGUMENT;
-    if (a.taps < 0 || (a.taps > 0 && (a.conv_w == nullptr || a.cu_seqlens == nullptr || a.slots == nullptr))) return MF_ERR_ARGUMENT;
+    if (a.taps < 0 || (a.taps > 0 && (a.conv_wt == nullptr || a.cu_seqlens == nullptr || a.slots == nullptr))) return MF_ERR_ARGUMENT;
     if (a.taps > 1 && a.conv_state == nullptr) return MF_ERR_ARGUMENT;
     if (head_run_fits(a)) {
         if (dtype == MF_DTYPE_F32) return head_run_launch<float>(a, n_tokens, stream);

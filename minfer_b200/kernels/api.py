@@ -1615,7 +1615,7 @@ class _HeadPrepArgs(ctypes.Structure):
                 [(n, c_int) for n in ("table_stride", "ring", "q_off", "n_heads", "qw", "k_off", "n_kv",
                                       "kw", "v_off", "vw", "rot_dims", "rot_style")] +
                 [(n, c_float) for n in ("rot_mag", "eps", "q_mul", "k_mul")] + [("status", c_void_p)] +
-                [(n, c_void_p) for n in ("conv_w", "conv_state", "cu_seqlens", "slots")] +
+                [(n, c_void_p) for n in ("conv_wt", "conv_state", "cu_seqlens", "slots")] +
                 [(n, c_int) for n in ("taps", "single")])
 
 
@@ -1636,7 +1636,7 @@ def head_prepare(proj: torch.Tensor, positions: torch.Tensor, token_row: torch.T
     ``v_off``) copied.  Writes q, the step's k and v and the cache's pages (each optional except q),
     in the type of ``q_out``.
 
-    ``conv`` (weight [channels, taps], state [slots, channels, taps - 1], cu_seqlens, slots, rows, whether
+    ``conv`` (weight [channels, taps], the same as [taps, channels], state [slots, channels, taps - 1], cu_seqlens, slots, rows, whether
     every row brings one token): a causal convolution without an activation over every channel of
     q | k | v (which lie side by side then) before all that, by this kernel where it takes the sizes, else
     by ``conv_silu``'s."""
@@ -1673,12 +1673,12 @@ def head_prepare(proj: torch.Tensor, positions: torch.Tensor, token_row: torch.T
     a.rot_mag, a.eps, a.q_mul, a.k_mul = float(rot_magnitude), float(eps), float(q_mul), float(k_mul)
     a.status = _i32(status, "status")
     if conv is not None:
-        weight, state, cu_seqlens, slots, n_rows, single = conv
+        weight, weight_t, state, cu_seqlens, slots, n_rows, single = conv
         channels, taps = weight.shape
         if (channels != n_heads * q_width + n_kv * (k_width + v_width) or k_off != q_off + n_heads * q_width
-                or v_off != k_off + n_kv * k_width or (taps > 1 and state.shape[1:] != (channels, taps - 1))):
+                or v_off != k_off + n_kv * k_width or weight_t.shape != (taps, channels) or (taps > 1 and state.shape[1:] != (channels, taps - 1))):
             raise KernelError("head_prepare: the convolution does not fit the heads")
-        a.conv_w, a.conv_state, a.taps = _f32(weight, "conv"), _f32(state, "conv state"), taps
+        a.conv_wt, a.conv_state, a.taps = _f32(weight_t, "conv"), _f32(state, "conv state"), taps
         a.cu_seqlens, a.slots, a.single = _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), 1 if single else 0
         if not _lib("mixer_prep").mf_head_prepare_takes_conv(ctypes.addressof(a)):
             u = torch.empty((n, channels), dtype=torch.float32, device=proj.device)

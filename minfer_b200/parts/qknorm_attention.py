@@ -92,6 +92,7 @@ class QkNormAttention(Mixer):
         self.values = values
         self.conv = int(conv)
         self.conv_w: Optional[torch.Tensor] = None         # [channels, taps]: q | k | v
+        self.conv_wt: Optional[torch.Tensor] = None        # the same as [taps, channels]
         self.names = "qk" if values == "keys" else "qkv"   # the projections' tensors
         self.out_scale = float(out_scale)
         self.tensor_prefix = tensor_prefix
@@ -143,6 +144,7 @@ class QkNormAttention(Mixer):
         self.out = Linear(weights[f"{p}o"])
         if self.conv:
             self.conv_w = torch.cat([weights[f"{p}{n}.conv"] for n in self.names], dim=0).contiguous()
+            self.conv_wt = self.conv_w.t().contiguous()
         if self.qk_norm:
             self.q_norm, self.k_norm = weights[f"{p}q.norm"], weights[f"{p}k.norm"]
         # the projection of q|k|v can apply a norm's 1/rms itself (bfloat16 on tensor cores)
@@ -210,7 +212,7 @@ class QkNormAttention(Mixer):
             state = binding.state.get(CONV_STATE)
             if state is None:        # one tap: nothing is kept
                 state = torch.empty((1, channels, 0), dtype=torch.float32, device=dev)
-            conv = (self.conv_w, state, ctx.cu_seqlens, ctx.slots, ctx.n_rows, ctx.single_token)
+            conv = (self.conv_w, self.conv_wt, state, ctx.cu_seqlens, ctx.slots, ctx.n_rows, ctx.single_token)
             if self.norm_scope == "all" or self.values == "keys":
                 # the kernel that prepares head by head convolves as it reads; here it comes first
                 heads = torch.empty((n, channels), dtype=torch.float32, device=dev)

@@ -388,7 +388,7 @@ def test_heads_behind_a_convolution(nh, nk, qw, vw, rot, style, taps, dt, lens):
         n = x.shape[0]
         proj = torch.cat([torch.randn(n, off, generator=g), x, torch.randn(n, 4, generator=g)], 1).to(DEV)
         outs = [torch.empty(n, h, w, dtype=dt, device=DEV) for h, w in ((nh, qw), (nk, qw), (nk, vw))]
-        conv = (cw.to(DEV), state, _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), len(rows), max(take) == 1) if taps else None
+        conv = (cw.to(DEV), cw.t().contiguous().to(DEV), state, _i32(_cu(take)), _i32([SLOTS[b] for b in rows]), len(rows), max(take) == 1) if taps else None
         K.head_prepare(proj, _i32([f + i for f, t in zip(first, take) for i in range(t)]),
                        _i32([i for i, t in enumerate(take) for _ in range(t)]), _i32([f + t for f, t in zip(first, take)]),
                        *outs, kc, vc, order[rows].int().to(DEV).contiguous(), pages, 0, q_off=off, n_heads=nh, q_width=qw,
