@@ -971,7 +971,8 @@ extern "C" int mf_head_prepare(const HeadPrepArgs* args, int n_tokens, int dtype
     if (a.k_cache != nullptr && a.page_table == nullptr) return MF_ERR_ARGUMENT;
     if (a.taps < 0 || (a.taps > 0 && (a.conv_wt == nullptr || a.cu_seqlens == nullptr || a.slots == nullptr))) return MF_ERR_ARGUMENT;
     if (a.taps > 1 && a.conv_state == nullptr) return MF_ERR_ARGUMENT;
-    if (head_run_fits(a)) {
+    // (without a convolution the float32 engine stays with the element-by-element form)
+    if (head_run_fits(a) && (a.taps > 0 || dtype != MF_DTYPE_F32)) {
         if (dtype == MF_DTYPE_F32) return head_run_launch<float>(a, n_tokens, stream);
         if (dtype == MF_DTYPE_BF16) return head_run_launch<__nv_bfloat16>(a, n_tokens, stream);
         return MF_ERR_UNSUPPORTED;

@@ -1772,9 +1772,11 @@ extern "C" int mf_norm_terms(const NormTermsArgs* args, int n_rows, int out_dtyp
     const bool vec = (a.width & 3) == 0 && (ptrs & 15) == 0;
     const int per = vec ? 4 : 1;
     if (a.width > 4 * 1024 * per) return MF_ERR_UNSUPPORTED;
-    // (a function of the width only: a row's sums never depend on the batch)
+    // (a function of the width and of the terms' form only: a row's sums never depend on the rows beside it.
+    // K splits come with few rows, whose loads then want as many threads as there are groups)
+    const bool wide = a.t1.n_part > 0 || a.t2.n_part > 0;
     int threads = 32;
-    while (threads < 1024 && threads * 2 * per < a.width) threads <<= 1;
+    while (threads < 1024 && threads * (wide ? 1 : 2) * per < a.width) threads <<= 1;
 #define MF_NT2(T, V, P) mf_launch(norm_terms_kernel<T, V, P>, dim3(n_rows), dim3(threads), 0, stream, a)
 #define MF_NT(T, V) do { if (pair) MF_NT2(T, V, true); else MF_NT2(T, V, false); } while (0)
     if (out_dtype == MF_DTYPE_F32) { if (vec) MF_NT(float, 4); else MF_NT(float, 1); }
